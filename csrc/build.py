@@ -5,7 +5,10 @@ linking, so the compiler can allocate registers per warp-specialised branch; the
 translation unit, folded on the host) and linked into one shared library.  Objects are rebuilt only when their source
 or a header under ``csrc/common`` is newer.
 
-    python csrc/build.py [--force] [--verbose]
+``--component serve`` builds only what inference of the decoder families needs (no gradients, no collectives) into
+``libdptb200_serve.so``.
+
+    python csrc/build.py [--force] [--verbose] [--component serve]
 """
 from __future__ import annotations
 
@@ -29,6 +32,11 @@ NVCC_FLAGS = [
     f"-I{CSRC}",
 ]
 
+COMPONENTS = {
+    "serve": ["gemm", "gemm_nt", "gemm_skinny", "gemm_grouped", "attention_fwd", "latent_attention", "recurrent",
+              "moe_local", "stream_norm", "elementwise"],
+}
+
 
 def nvcc_path() -> str:
     for cand in (os.environ.get("NVCC"), "/usr/local/cuda/bin/nvcc", "nvcc"):
@@ -37,7 +45,9 @@ def nvcc_path() -> str:
     return "nvcc"
 
 
-def sources():
+def sources(component=None):
+    if component is not None:
+        return [CSRC / f"{name}.cu" for name in COMPONENTS[component]]
     return sorted(CSRC.glob("*.cu"))
 
 
@@ -60,12 +70,13 @@ def _compile(src: Path, force: bool, verbose: bool, hdr_mtime: float):
     return obj, True, proc.stderr
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def build(force: bool = False, verbose: bool = False, component=None) -> Path:
+    lib = LIB if component is None else LIB.with_name(LIB.name.replace(".so", f"_{component}.so"))
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
     OUT_DIR.mkdir(parents=True, exist_ok=True)
     hdr_mtime = _newest_header_mtime()
-    srcs = sources()
-    with ThreadPoolExecutor(max_workers=min(8, max(1, len(srcs)))) as pool:
+    srcs = sources(component)
+    with ThreadPoolExecutor(max_workers=min(max(8, os.cpu_count() or 1), max(1, len(srcs)))) as pool:
         results = list(pool.map(lambda s: _compile(s, force, verbose, hdr_mtime), srcs))
     objs = [r[0] for r in results]
     rebuilt = any(r[1] for r in results)
@@ -73,21 +84,22 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         for r in results:
             if r[2]:
                 print(r[2])
-    stale = (not LIB.exists()) or any(o.stat().st_mtime > LIB.stat().st_mtime for o in objs)
+    stale = (not lib.exists()) or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs)
     if rebuilt or stale or force:
-        cmd = [nvcc_path(), "-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-o", str(LIB),
+        cmd = [nvcc_path(), "-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-o", str(lib),
                *[str(o) for o in objs], "-Xcompiler", "-fPIC"]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         if proc.returncode != 0:
             raise RuntimeError(f"link failed:\n{proc.stdout}\n{proc.stderr}")
-    return LIB
+    return lib
 
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true")
+    ap.add_argument("--component", choices=sorted(COMPONENTS), default=None)
     args = ap.parse_args()
-    lib = build(args.force, args.verbose)
+    lib = build(args.force, args.verbose, args.component)
     print(lib)
     sys.exit(0)

@@ -35,6 +35,18 @@ class KernelError(RuntimeError):
 
 
 LIB_NAME = "libdptb200.so"
+_COMPONENT: Optional[str] = None      # a subset of the kernels that is enough for this process (see csrc/build.py)
+
+
+def use_component(name: Optional[str]) -> None:
+    """Where the whole library has not been built, the component library ``libdptb200_<name>.so`` may stand in for it in
+    this process (and is what an automatic build compiles)."""
+    global _COMPONENT
+    _COMPONENT = name
+
+
+def component_lib_name(name: str) -> str:
+    return LIB_NAME.replace(".so", f"_{name}.so")
 
 
 def candidate_paths() -> list:
@@ -49,6 +61,8 @@ def candidate_paths() -> list:
     if sys.argv and sys.argv[0]:
         out.append(Path(sys.argv[0]).resolve().parent / LIB_NAME)
     out.append(_HERE / "_C" / LIB_NAME)
+    if _COMPONENT:
+        out.append(_HERE / "_C" / component_lib_name(_COMPONENT))
     return out
 
 
@@ -71,8 +85,9 @@ def build_native_library() -> Optional[Path]:
     script = _HERE.parent / "csrc" / "build.py"
     if os.environ.get("DPTB200_AUTO_BUILD", "0") != "1" or not script.exists() or shutil.which("nvcc") is None:
         return None
-    subprocess.run([sys.executable, str(script)], check=True)
-    built = _HERE / "_C" / LIB_NAME
+    extra = ["--component", _COMPONENT] if _COMPONENT else []
+    subprocess.run([sys.executable, str(script), *extra], check=True, stdout=sys.stderr)
+    built = _HERE / "_C" / (component_lib_name(_COMPONENT) if _COMPONENT else LIB_NAME)
     return built if looks_like_shared_object(built) else None
 
 

@@ -32,13 +32,16 @@ from ..coop.http_coop import ServerHandle
 # -------------------------------------------------------------------------------------------- model loading --
 def load_hf_model(family: str, model_dir: str, device=None, dtype=torch.float32, preset: Optional[str] = None):
     """Build and load a causal LM from ``<model_dir>/model.safetensors`` (or a sharded index) and, when present,
-    ``tokenizer.json``.  ``family``: ``gpt2``, ``distilgpt2``, ``pythia``, ``gptj`` or ``llama``; ``preset`` picks the size
-    (e.g. ``medium``, ``160m``, ``8b``); without one the size is inferred from the checkpoint's tensor shapes."""
+    ``tokenizer.json``.  ``family``: ``gpt2``, ``distilgpt2``, ``pythia``, ``gptj``, ``llama``, ``famudra`` or ``auto`` (the
+    family that ``config.json`` names); ``preset`` picks the size (e.g. ``medium``, ``160m``, ``8b``); without one the size is
+    inferred from the checkpoint's tensor shapes (``famudra``: read from ``config.json``)."""
     from ..data.hf_tokenizers import HFBpeTokenizer
     from ..io.hf_loaders import GPT2HFLoader, LlamaHFLoader
     from ..io.hf_loaders_more import GPTJHFLoader, PythiaHFLoader
     from ..io.safetensors import SafeTensors
-    from ..models import GPT, GPTJModel, Llama, PythiaModel
+    from ..models import GPT, GPTJModel, Llama, PythiaModel, registry
+    if family.lower() == "auto":
+        family = registry.family_of(registry.read_config(model_dir))
     idx = os.path.join(model_dir, "model.safetensors.index.json")
     state = SafeTensors.load_sharded(idx) if os.path.exists(idx) else SafeTensors.load_file(
         os.path.join(model_dir, "model.safetensors"))
@@ -70,6 +73,10 @@ def load_hf_model(family: str, model_dir: str, device=None, dtype=torch.float32,
             preset = {2048: "1b", 3072: "3b", 4096: "8b"}[d]
         model = Llama(presets[preset](**kw))
         report = LlamaHFLoader.load_map(model, state)
+    elif fam in registry.ARCHITECTURES:
+        arch = registry.architecture(fam)
+        model = arch.build(registry.read_config(model_dir), **kw)
+        report = arch.load_map(model, state)
     else:
         raise ValueError(f"unknown model family {family!r}")
     tok_path = os.path.join(model_dir, "tokenizer.json")

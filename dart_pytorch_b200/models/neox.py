@@ -29,9 +29,22 @@ from .gpt import GPT, _as_token_tensor
 class CausalLMMixin:
     """Sampling loop shared by the decoder-only families: needs ``self.config.{max_ctx, vocab_size}``,
     ``self.logits(tokens, start_pos, cache)`` and ``self.new_cache()`` (reference: lib/core/nn/gpt.dart:185-342 —
-    the other families repeat that loop verbatim)."""
+    the other families repeat that loop verbatim).  A family may compute only the last position (``last_logits``) and may
+    pool its caches (``free_cache``)."""
 
     _name = "Model"
+
+    def last_logits(self, tokens, start_pos: int = 0, cache=None):
+        """Logits after the last token of every sequence: ``[1, V]`` for ``[N]`` tokens, ``[B, V]`` for ``[B, N]``."""
+        out = self.logits(tokens, start_pos, cache)
+        return out[-1:] if out.dim() == 2 else out[:, -1]
+
+    def cache_for(self, tokens: int):
+        """A new cache for one sequence of up to ``tokens`` tokens (families with a fixed context size it by that)."""
+        return self.new_cache()
+
+    def free_cache(self, cache) -> None:
+        """The sequences of this cache are finished."""
 
     def generate(self, prompt: Sequence[float], max_new_tokens: int, temperature: float = 1.0,
                  top_k: Optional[int] = None, rng=None, use_cache: bool = True,
@@ -51,24 +64,52 @@ class CausalLMMixin:
                 out = [float(t) for t in prompt]
                 sample = lambda row: GPT._sample(self, row, temperature, top_k, rng)  # noqa: E731
                 if use_cache:
-                    cache = self.new_cache()
-                    logits = self.logits(_as_token_tensor(prompt, self.input_device), 0, cache)
-                    nxt = sample(logits[-1])
+                    cache = self.cache_for(min(c.max_ctx, len(prompt) + max_new_tokens))
+                    nxt = sample(self.last_logits(_as_token_tensor(prompt, self.input_device), 0, cache)[0])
                     out.append(float(nxt))
                     for _ in range(1, max_new_tokens):
                         if cache.seq_len >= c.max_ctx or (stop_id is not None and nxt == stop_id):
                             break
                         tok = torch.tensor([nxt], dtype=torch.long, device=self.input_device)
-                        nxt = sample(self.logits(tok, cache.seq_len, cache)[-1])
+                        nxt = sample(self.last_logits(tok, cache.seq_len, cache)[0])
                         out.append(float(nxt))
+                    self.free_cache(cache)
                 else:
                     for _ in range(max_new_tokens):
                         ctx = out[-c.max_ctx:]
-                        nxt = sample(self.logits(_as_token_tensor(ctx, self.input_device), 0, None)[-1])
+                        nxt = sample(self.last_logits(_as_token_tensor(ctx, self.input_device), 0, None)[0])
                         out.append(float(nxt))
                         if stop_id is not None and nxt == stop_id:
                             break
                 return out
+        finally:
+            if was_training:
+                self.train()
+
+    def generate_batch(self, prompts: torch.Tensor, max_new_tokens: int) -> torch.Tensor:
+        """Greedy decoding of a ``[B, N]`` batch of equal-length prompts with device argmax; returns ``[B, N + new]`` token
+        ids.  Nothing but the final ids leaves the device.  Needs ``new_cache(max_len, batch)``."""
+        was_training = self.training
+        self.eval()
+        try:
+            with torch.no_grad():
+                toks = _as_token_tensor(prompts, self.input_device)
+                B, n = toks.shape
+                cache = self.new_cache(min(self.config.max_ctx, n + max_new_tokens), B)
+                outs, cur = [toks], toks
+                for step in range(max_new_tokens):
+                    logits = self.last_logits(cur, cache.seq_len, cache)
+                    if logits.is_cuda:
+                        from ..ops import kernels as K
+                        nxt = K.argmax_rows(logits, n_cols=self.config.vocab_size)
+                    else:
+                        nxt = logits.argmax(-1)
+                    cur = nxt.reshape(B, 1)
+                    outs.append(cur)
+                    if step + 1 == max_new_tokens or cache.seq_len >= self.config.max_ctx:
+                        break
+                self.free_cache(cache)
+                return torch.cat(outs, dim=1)
         finally:
             if was_training:
                 self.train()
