@@ -19,6 +19,9 @@
 // The output accumulator never leaves TMEM during the loop.  The running maximum is lazy: a row keeps exponentiating
 // against an older maximum until the true one has grown by more than 8 (a factor 256 of headroom in fp32 / bf16);
 // only then (decided per warp) O is pulled out, rescaled and stored back, which after the first tiles is rare.
+//
+// The precise form (PREC) walks tiles of 64 keys and keeps every softmax weight as a high and a low bf16 part (16 mantissa
+// bits): both parts of a 64-key tile take the room one part of a 128-key tile has, and P V is two products.
 #include <cuda_bf16.h>
 
 #include "common/host.h"
@@ -44,7 +47,6 @@ __device__ __forceinline__ float fast_exp2(float x) {
 }
 
 constexpr int kAttnBM = 128;   // query rows per tile
-constexpr int kAttnBN = 128;   // keys per tile
 constexpr int kAttnThreads = 384;   // two softmax warpgroups + one warpgroup holding the TMA and MMA warps
 // Registers per thread after the hand-over.  The CTA starts with 384 x 168 registers and the pool does not grow:
 // 2 x 128 x 216 + 128 x 72 = 384 x 168, so the increase can always be satisfied once the producers have shrunk.
@@ -65,11 +67,12 @@ __device__ unsigned long long g_attn_prof[8];
 #define ATTN_PROF_ADD(slot, t0, t1)
 #endif
 
-template <int HD, int NQ, int KST, int VST>
+template <int HD, int NQ, int KST, int VST, bool PREC>
 struct AttnFwdSmem {
+  static constexpr int kBN = PREC ? 64 : 128;           // keys per tile
   static constexpr int kQBytes = kAttnBM * HD * 2;
-  static constexpr int kKVBytes = kAttnBN * HD * 2;
-  static constexpr int kPBytes = kAttnBM * kAttnBN * 2;
+  static constexpr int kKVBytes = kBN * HD * 2;
+  static constexpr int kPBytes = kAttnBM * 128 * 2;     // 128 keys, or 64 keys twice
   static constexpr int kQOff = 0;
   static constexpr int kKOff = kQOff + NQ * kQBytes;
   static constexpr int kVOff = kKOff + KST * kKVBytes;
@@ -80,11 +83,12 @@ struct AttnFwdSmem {
   static_assert(kTotal <= 227 * 1024, "attention forward: shared memory budget");
 };
 
-template <int HD, int NQ, int KST, int VST>
+template <int HD, int NQ, int KST, int VST, bool PREC>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, const AttnFwdParams p) {
-  using L = AttnFwdSmem<HD, NQ, KST, VST>;
+  using L = AttnFwdSmem<HD, NQ, KST, VST, PREC>;
+  constexpr int kAttnBN = L::kBN;
   constexpr int kChunks = HD / 64;            // 64-column (128-byte) chunks per head row
   constexpr int TMEM_COLS = 512;
   constexpr int kSCol = 0;                    // S_t at columns [t*128, t*128+128)
@@ -217,9 +221,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         const uint32_t kb = smem_u32(smem + L::kKOff + (j % KST) * L::kKVBytes);
 #pragma unroll
         for (int kk = 0; kk < HD / 16; ++kk) {
-          const uint32_t off = (kk / 4) * (kAttnBM * 128) + (kk % 4) * 32;
-          umma_bf16(tmem_base + kSCol + t * kAttnBN, make_smem_desc(qa + off, 16, 1024),
-                    make_smem_desc(kb + off, 16, 1024), idesc_s, kk != 0);
+          const uint32_t q_off = (kk / 4) * (kAttnBM * 128) + (kk % 4) * 32;
+          const uint32_t k_off = (kk / 4) * (kAttnBN * 128) + (kk % 4) * 32;
+          umma_bf16(tmem_base + kSCol + t * 128, make_smem_desc(qa + q_off, 16, 1024),
+                    make_smem_desc(kb + k_off, 16, 1024), idesc_s, kk != 0);
         }
         umma_commit(&s_full[t]);
         issued_any = true;
@@ -262,10 +267,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           const uint32_t pa = smem_u32(smem + L::kPOff + t * L::kPBytes);
           const uint32_t vb = smem_u32(smem + L::kVOff + vs * L::kKVBytes);
 #pragma unroll
-          for (int kk = 0; kk < kAttnBN / 16; ++kk) {
+          for (int kk = 0; kk < 8; ++kk) {     // 128 keys, or the high and then the low parts of 64
             const uint32_t aoff = (kk / 4) * (kAttnBM * 128) + (kk % 4) * 32;
             umma_bf16(tmem_base + kOCol + t * HD, make_smem_desc(pa + aoff, 16, 1024),
-                      make_smem_desc(vb + kk * 2048, kAttnBN * 128, 1024), idesc_o, (j != 0 || kk != 0) ? 1u : 0u);
+                      make_smem_desc(vb + (PREC ? kk % 4 : kk) * 2048, kAttnBN * 128, 1024), idesc_o,
+                      (j != 0 || kk != 0) ? 1u : 0u);
           }
           umma_commit(&o_full[t]);
           issued_any = true;
@@ -289,7 +295,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const int q_row = q_row0 + t * kAttnBM + row_in_tile;         // row inside the sequence
     const int n = n_tiles[t];
     const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16);
-    const uint32_t s_addr = lane_addr + kSCol + t * kAttnBN;
+    const uint32_t s_addr = lane_addr + kSCol + t * 128;
     const uint32_t o_addr = lane_addr + kOCol + t * HD;
     uint8_t* p_tile = smem + L::kPOff + t * L::kPBytes;
 
@@ -368,7 +374,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       float l0 = 0.0f, l1 = 0.0f, l2 = 0.0f, l3 = 0.0f;
 #pragma unroll
       for (int c = 0; c < kAttnBN / 32; ++c) {
-        uint32_t packed[16];
+        uint32_t packed[16], low[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
           // (Computing half of the exponentials as cubic polynomials on the FMA pipe was measured slower here: 117 us
@@ -382,6 +388,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           l0 += a; l1 += b; l2 += e; l3 += f;
           packed[(i >> 1) + 0] = pack_bf16x2(a, b);
           packed[(i >> 1) + 1] = pack_bf16x2(e, f);
+          if constexpr (PREC) {
+            const float2 ab = unpack_bf16x2(packed[(i >> 1) + 0]), ef = unpack_bf16x2(packed[(i >> 1) + 1]);
+            low[(i >> 1) + 0] = pack_bf16x2(a - ab.x, b - ab.y);
+            low[(i >> 1) + 1] = pack_bf16x2(e - ef.x, f - ef.y);
+          }
         }
         // 32 keys = 64 bytes = four 16-byte chunks of this row, in 64-key block (c / 2), at chunk (c % 2) * 4 + i.
         uint8_t* blk = p_tile + (c >> 1) * (kAttnBM * 128);
@@ -390,6 +401,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           const uint32_t chunk = (uint32_t)((c & 1) * 4 + i) ^ (uint32_t)(row_in_tile & 7);
           *reinterpret_cast<uint4*>(blk + row_in_tile * 128 + chunk * 16) =
               make_uint4(packed[i * 4 + 0], packed[i * 4 + 1], packed[i * 4 + 2], packed[i * 4 + 3]);
+          if constexpr (PREC)
+            *reinterpret_cast<uint4*>(blk + kAttnBM * 128 + row_in_tile * 128 + chunk * 16) =
+                make_uint4(low[i * 4 + 0], low[i * 4 + 1], low[i * 4 + 2], low[i * 4 + 3]);
         }
       }
       l_run += (l0 + l1) + (l2 + l3);
@@ -479,11 +493,13 @@ struct DptbAttnFwdArgs {
   int causal, q_offset;
   float scale;
   long long kv_batch_rows;  // rows between consecutive batches of K / V (a cache's capacity); 0 = Sk
+  int precise;              // softmax weights as two bf16 parts
 };
 
-template <int HD, int NQ, int KST, int VST>
+template <int HD, int NQ, int KST, int VST, bool PREC>
 static int attn_fwd_launch(const DptbAttnFwdArgs* a, cudaStream_t st) {
-  using L = AttnFwdSmem<HD, NQ, KST, VST>;
+  using L = AttnFwdSmem<HD, NQ, KST, VST, PREC>;
+  constexpr int kAttnBN = L::kBN;
   CUtensorMap tmQ, tmK, tmV;
   int rc = encode_tmap_seq(&tmQ, a->q, a->Hq, HD, a->Sq, a->B, a->ldq, kAttnBM);
   if (rc) return rc;
@@ -500,7 +516,7 @@ static int attn_fwd_launch(const DptbAttnFwdArgs* a, cudaStream_t st) {
   p.q_offset = a->q_offset;
   p.scale_log2 = a->scale * 1.4426950408889634f;
   p.num_q_blocks = (a->Sq + NQ * kAttnBM - 1) / (NQ * kAttnBM);
-  auto kern = attn_fwd_kernel<HD, NQ, KST, VST>;
+  auto kern = attn_fwd_kernel<HD, NQ, KST, VST, PREC>;
   DPTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal));
   dim3 grid(p.num_q_blocks, a->Hq, a->B);
   kern<<<grid, kAttnThreads, L::kTotal, st>>>(tmQ, tmK, tmV, p);
@@ -526,7 +542,12 @@ extern "C" int dptb_attn_fwd(const DptbAttnFwdArgs* a, void* stream) {
   if (a->Sk <= 0 || a->Hkv <= 0 || a->Hq % a->Hkv) return kErrBadShape;
   if ((a->ldq % 8) || (a->ldk % 8) || (a->ldv % 8) || (a->ldo % 8)) return kErrBadShape;
   if ((reinterpret_cast<uintptr_t>(a->o) & 15) != 0) return kErrBadShape;
-  if (a->head_dim == 64) return attn_fwd_launch<64, 2, 2, 2>(a, st);
-  if (a->head_dim == 128) return attn_fwd_launch<128, 2, 2, 1>(a, st);
+  if (a->precise) {
+    if (a->head_dim == 64) return attn_fwd_launch<64, 2, 4, 4, true>(a, st);
+    if (a->head_dim == 128) return attn_fwd_launch<128, 2, 3, 3, true>(a, st);
+    return kErrUnsupported;
+  }
+  if (a->head_dim == 64) return attn_fwd_launch<64, 2, 2, 2, false>(a, st);
+  if (a->head_dim == 128) return attn_fwd_launch<128, 2, 2, 1, false>(a, st);
   return kErrUnsupported;
 }

@@ -132,8 +132,9 @@ struct LruChannel {
     bi = to_f32(static_cast<const T*>(p.bi)[ch]);
     decay = -p.c * softplus_f(to_f32(static_cast<const T*>(p.lam)[ch]));
   }
-  // log decay and input of token t
-  __device__ __forceinline__ void step(int t, float& log_a, float& in) const {
+  // Applies token t to S; returns its log decay.  With e = a - 1 = expm1(log a), which keeps its relative precision where
+  // a is next to 1:  1 - a^2 = -e (2 + e)  and  a S = S + e S, so long memories do not drift.
+  __device__ __forceinline__ float step(int t, float& S) const {
     const float* zt = z + (long long)t * 2 * C;
     float uv;
     if constexpr (sizeof(T) == 2) {
@@ -142,8 +143,10 @@ struct LruChannel {
     } else {
       uv = to_f32(u[(long long)t * C]);
     }
-    log_a = decay * sigmoid_f(zt[0] + br);
-    in = sqrtf(-expm1f(2.0f * log_a)) * sigmoid_f(zt[bw] + bi) * uv;
+    const float log_a = decay * sigmoid_f(zt[0] + br);
+    const float e = expm1f(log_a);
+    S += fmaf(e, S, sqrtf(-e * (2.0f + e)) * sigmoid_f(zt[bw] + bi) * uv);
+    return log_a;
   }
 };
 
@@ -164,10 +167,7 @@ __global__ void __launch_bounds__(128) lru_chunk_kernel(const LruParams p) {
   const int t0 = k * p.chunk, t1 = t0 + p.chunk;
 #pragma unroll 4
   for (int t = t0; t < t1; ++t) {
-    float la, in;
-    lc.step(t, la, in);
-    total += la;
-    S = fmaf(expf(la), S, in);
+    total += lc.step(t, S);
   }
   agg[(long long)k * 2 * p.C] = total;
   agg[((long long)k * 2 + 1) * p.C] = S;
@@ -191,7 +191,8 @@ __global__ void __launch_bounds__(128) lru_scan_kernel(const LruParams p) {
     } else {
       S = agg[p.C];
 #pragma unroll 4
-      for (int j = 1; j < k; ++j) S = fmaf(expf(agg[(long long)j * 2 * p.C]), S, agg[((long long)j * 2 + 1) * p.C]);
+      for (int j = 1; j < k; ++j)
+        S += fmaf(expm1f(agg[(long long)j * 2 * p.C]), S, agg[((long long)j * 2 + 1) * p.C]);
     }
   }
   const int t0 = k * p.chunk, t1 = min(p.S, t0 + p.chunk);
@@ -199,9 +200,7 @@ __global__ void __launch_bounds__(128) lru_scan_kernel(const LruParams p) {
   T* out = static_cast<T*>(p.out) + (long long)b * p.S * p.C + ch;
 #pragma unroll 4
   for (int t = t0; t < t1; ++t) {
-    float la, in;
-    lc.step(t, la, in);
-    S = fmaf(expf(la), S, in);
+    lc.step(t, S);
     out[(long long)t * p.C] = from_f32<T>(S * gelu_tanh_f(to_f32(y[(long long)t * p.ldy])));
   }
   if (k == p.chunks - 1) p.state[(long long)b * p.C + ch] = S;

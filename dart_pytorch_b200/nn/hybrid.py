@@ -308,7 +308,7 @@ class LatentAttention(_Packed):
         else:
             kv = torch.cat([F.linear(state.buf[b, :n], pack["ukv"]) for b in range(B)], 0)
         o, _ = flash.attn_fwd(q, kv[:, :H * pd], kv[:, H * pd:], B, S, n, H, H, pd, True, q_offset=ctx.pos,
-                              scale=self.scale, need_lse=False)
+                              scale=self.scale, need_lse=False, precise=True)
         return F.linear(o, pack["wo"])
 
 

@@ -24,7 +24,7 @@ class AttnFwdArgs(ctypes.Structure):
     _fields_ = [("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("o", c_void_p), ("lse", c_void_p),
                 ("ldq", c_ll), ("ldk", c_ll), ("ldv", c_ll), ("ldo", c_ll),
                 ("B", c_int), ("Sq", c_int), ("Sk", c_int), ("Hq", c_int), ("Hkv", c_int), ("head_dim", c_int),
-                ("causal", c_int), ("q_offset", c_int), ("scale", c_float), ("kv_batch_rows", c_ll)]
+                ("causal", c_int), ("q_offset", c_int), ("scale", c_float), ("kv_batch_rows", c_ll), ("precise", c_int)]
 
 
 class AttnBwdArgs(ctypes.Structure):
@@ -84,8 +84,9 @@ def _ld(t: torch.Tensor) -> int:
 
 
 def attn_fwd(q2, k2, v2, B, Sq, Sk, Hq, Hkv, hd, causal, q_offset=0, scale=None, need_lse=True, out=None,
-             kv_batch_rows=0):
-    """Forward kernel call on token-major 2-D views (``q2``: ``[B*Sq, >= Hq*hd]`` etc.).  Returns ``(o, lse)``."""
+             kv_batch_rows=0, precise=False):
+    """Forward kernel call on token-major 2-D views (``q2``: ``[B*Sq, >= Hq*hd]`` etc.).  Returns ``(o, lse)``.
+    ``precise`` keeps the softmax weights in two bf16 parts (16 mantissa bits) for the product with V."""
     lib = N.load()
     if out is None:
         out = torch.empty(B * Sq, Hq * hd, dtype=torch.bfloat16, device=q2.device)
@@ -97,6 +98,7 @@ def attn_fwd(q2, k2, v2, B, Sq, Sk, Hq, Hkv, hd, causal, q_offset=0, scale=None,
     a.causal, a.q_offset = int(causal), int(q_offset)
     a.scale = (1.0 / math.sqrt(hd)) if scale is None else scale
     a.kv_batch_rows = kv_batch_rows
+    a.precise = int(precise)
     N.check(lib.dptb_attn_fwd(ctypes.byref(a), N.stream_ptr()), "attn_fwd")
     return out, lse
 

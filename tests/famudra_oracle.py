@@ -112,6 +112,69 @@ def moe(h, w, mlp):
     return out
 
 
+def shapes(config):
+    """``{tensor name: shape}`` of a model."""
+    D = config["width"]
+    out = {"embed": [config["vocab"], D], "final.norm": [], "head": [config["vocab"], D]}
+    for i, spec in enumerate(config["layers"]):
+        m, mlp = spec["mixer"], spec["mlp"]
+        s = {"norm1": [], "shift": [D]}
+        if spec["type"] == "rglru":
+            C, G = m["width"], m["blocks"]
+            n = C // G
+            s.update({"mix.y": [C, D], "mix.y.b": [C], "mix.x": [C, D], "mix.x.b": [C], "mix.conv": [C, m["conv"]],
+                      "mix.conv.b": [C], "mix.ra": [G, n, n], "mix.ra.b": [G, n], "mix.ri": [G, n, n], "mix.ri.b": [G, n],
+                      "mix.lam": [C], "mix.o": [D, C]})
+        else:
+            H, R = m["heads"], m["kv_rank"]
+            s.update({"mix.dq": [m["q_rank"], D], "mix.dq.norm": [m["q_rank"]], "mix.dkv": [R, D], "mix.dkv.norm": [R],
+                      "mix.uq": [H * m["dim"], m["q_rank"]], "mix.uk": [H * m["dim"], R], "mix.uv": [H * m["vdim"], R],
+                      "mix.o": [D, H * m["vdim"]]})
+        if mlp:
+            s.update({"norm2": [], "mlp.router": [mlp["router"]["experts"], D]})
+            for e in range(mlp["router"]["experts"]):
+                s.update({f"mlp.e{e}.up": [mlp["expert"]["ff"], D], f"mlp.e{e}.down": [D, mlp["expert"]["ff"]]})
+            if mlp.get("shared"):
+                s.update({"mlp.shared.up": [mlp["shared"]["ff"], D], "mlp.shared.down": [D, mlp["shared"]["ff"]]})
+        out.update({f"l{i}.{k}": v for k, v in s.items()})
+    return out
+
+
+def random_weights(config, seed, gain=1.0):
+    """bf16-representable random weights that keep every branch's output of the order of the stream."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in shapes(config).items():
+        leaf = name.split(".", 1)[-1]
+        r = torch.randn(*shape, generator=g) if shape else torch.randn(1, generator=g).reshape(())
+        if not shape or leaf.endswith(".norm"):
+            t = 1.0 + 0.2 * r
+        elif name.endswith(".shift"):
+            t = torch.sigmoid(r)
+        elif name.endswith(".lam"):
+            t = -4.0 + 2.0 * r                       # decays between a few and thousands of tokens
+        elif len(shape) == 1 or leaf.endswith("ra.b") or leaf.endswith("ri.b"):
+            t = 0.3 * r
+        elif name == "embed":
+            t = r
+        elif leaf == "mix.conv":
+            t = 0.6 * r
+        elif leaf == "mlp.router":
+            t = 3.0 * r / math.sqrt(shape[-1])
+        else:
+            t = gain * r / math.sqrt(shape[-1])
+        out[name] = t.to(torch.bfloat16).float()
+    return out
+
+
+def greedy(config, weights, prompt, n, dtype=torch.float64):
+    """``prompt`` followed by ``n`` tokens of largest logit, every step from scratch."""
+    out = list(prompt)
+    for _ in range(n):
+        out.append(int(run(config, weights, out, dtype)[-1].argmax()))
+    return out
+
+
 def layer_schedule(config):
     """Layer indices in the order they run, each with a flag: the embedding output is added before it."""
     n = len(config["layers"])
