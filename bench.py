@@ -40,6 +40,9 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "torch"])
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--batch", type=int, default=MICRO_BATCH)
+    ap.add_argument("--workload", default="gpt2_train", choices=["gpt2_train", "famudra"],
+                    help="famudra: prompt and decode throughput of the hybrid decoder beside Llama at equal size, one GPU")
+    ap.add_argument("--sizes", default="small,medium,large", help="model sizes of the famudra workload")
     return ap.parse_args()
 
 
@@ -305,9 +308,18 @@ def run_reference(args):
     run(args, METRIC, MODEL, SEQ, ClockSampler)
 
 
+def run_famudra(args):
+    import torch
+    from benchmarks.hybrid_bench import bench_line
+    torch.cuda.set_device(0)
+    print(json.dumps(bench_line(args, ClockSampler)))
+
+
 if __name__ == "__main__":
     a = parse_args()
-    if a.impl == "reference":
+    if a.workload == "famudra":
+        run_famudra(a)
+    elif a.impl == "reference":
         run_reference(a)
     elif a.impl == "torch":
         run_torch(a)

@@ -171,6 +171,119 @@ def build_cases(dev, want=()):
         od = torch.empty(Bd, Hq * hdd, **bf)
         cases["attn_decode"] = (lambda: Dk.attn_decode(qd, kc, vc, Bd, 1, Sk, Hq, Hkv, hdd, Sk - 1, out=od),
                                 2 * 2 * Bd * Sk * Hkv * hdd, 0.0)
+    if on("hybrid"):
+        cases.update(build_hybrid_cases(dev))
+    return cases
+
+
+def build_hybrid_cases(dev):
+    """Serving kernels of the hybrid decoder (Famudra) at the "medium" size of ``hybrid_bench.py``, 4 x 2048 prompt tokens and
+    32 decode rows over 2304 tokens, and (``hybrid_like_*``) the kernels that play the same part in Llama at that width."""
+    from dart_pytorch_b200.nn.hybrid import DroplessMoE
+    from dart_pytorch_b200.ops import decode as Dk
+    from dart_pytorch_b200.ops import hybrid as Y
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    f32 = dict(device=dev, dtype=torch.float32)
+    D, H, hd, Rq, R, C, G, E, top, ff, sff, V = 2048, 16, 128, 768, 512, 2560, 10, 64, 6, 1024, 2048, 32768
+    B, S = 4, 2048
+    M, Bd, Sk = B * S, 32, 2304
+    rn = lambda *s: torch.randn(*s, **bf)  # noqa: E731
+    cases = {}
+
+    def add(name, fn, nbytes, flops=0.0):
+        cases["hybrid_" + name] = (fn, nbytes, flops)
+
+    def gemm(name, m, n, k):
+        a, w, c = rn(m, k), rn(n, k), torch.empty(m, n, **bf)
+        add(name, lambda: K.gemm(a, w, c, trans_b=True), 2 * (m * k + n * k + m * n), 2.0 * m * n * k)
+    # ---- prompts
+    gemm("like_gemm_gate_up", M, 2 * 5464 // 8 * 8, D)
+    gemm("gemm_dq_dkv", M, Rq + R, D)
+    q2, k2, v2, o2 = rn(M, H * hd), rn(M, H * hd), rn(M, H * hd), torch.empty(M, H * hd, **bf)
+    fl = 4.0 * B * H * S * S * hd / 2
+    for name, precise in (("like_attn_fwd", False), ("attn_fwd_precise", True)):
+        add(name, lambda precise=precise: A.attn_fwd(q2, k2, v2, B, S, S, H, H, hd, True, out=o2, need_lse=False,
+                                                     precise=precise), 2 * 4 * M * H * hd, fl)
+    moe = {}
+    for tag, rows in (("", M), ("dec_", Bd)):
+        m = DroplessMoE(8, E, top, 8, 0, device=dev, dtype=torch.bfloat16)
+        router, x = rn(E, D), rn(rows, D)
+        ctr = torch.zeros(2 * E, dtype=torch.int32, device=dev)
+        idx, w = Y.moe_route(x, router, top, ctr)
+        base = ctr.clone()
+        xs, off, slot = Y.moe_place(x, idx, ctr, E)
+        if tag == "":
+            wu, wd, su, sd = rn(E * ff, D), rn(E * D, ff), rn(sff, D), rn(D, sff)
+        up, y, s_up, sh = torch.empty(rows * top, ff, **bf), rn(rows * top, D), torch.empty(rows, sff, **bf), rn(rows, D)
+        hint = (rows * top + E - 1) // E
+        live = int((base[:E] > 0).sum())
+        seg = Y.grouped_segment
+
+        def run_up(x=x, xs=xs, up=up, off=off, s_up=s_up, hint=hint):
+            Y.grouped_gemm(seg(xs, wu, up, groups=E, N_=ff, K=D, offsets=off, act="relu2", rows_hint=hint),
+                           seg(x, su, s_up, groups=1, N_=sff, K=D, act="relu2"))
+
+        def run_down(up=up, y=y, off=off, s_up=s_up, sh=sh, hint=hint):
+            Y.grouped_gemm(seg(up, wd, y, groups=E, N_=D, K=ff, offsets=off, rows_hint=hint),
+                           seg(s_up, sd, sh, groups=1, N_=D, K=sff))
+        wb = 2 * (live * ff * D + sff * D)
+        flops = 2.0 * rows * D * (top * ff + sff)
+        add(tag + "experts_up", run_up, wb + 2 * rows * (top * (D + ff) + D + sff), flops)
+        add(tag + "experts_down", run_down, wb + 2 * rows * (top * (D + ff) + D + sff), flops)
+        add(tag + "route", lambda x=x, ctr=ctr: Y.moe_route(x, router, top, ctr), 2 * rows * D)
+
+        def place(x=x, idx=idx, ctr=ctr, base=base):
+            ctr.copy_(base)
+            Y.moe_place(x, idx, ctr, E)
+        add(tag + "place", place, 2 * rows * D * (1 + top))
+        xr, mix, g, mu, st = torch.randn(rows, D, **f32), rn(rows, D), rn(1), rn(D), torch.zeros(B if tag == "" else rows, D, **f32)
+        t = Y.LayerTerms(mix, sh, y, slot, w)
+        add(tag + "stream_norm", lambda xr=xr, t=t, rows=rows, g=g, mu=mu, st=st: Y.stream_norm(
+            xr, t, rows, rows // st.shape[0], g, 1e-6, g2=g, shift=mu, shift_state=st), rows * D * (4 + 2 + 2 + 2 * top + 4 + 4))
+        gamma = rn(D)
+        add("like_" + tag + "rmsnorm", lambda x=x, gamma=gamma: K.rmsnorm_fwd(x, gamma, 1e-5), 4 * rows * D)
+        # ---- recurrence
+        seqs = B if tag == "" else rows
+        n = C // G
+        yx, taps, bias = rn(rows, 2 * C), rn(C, 4), rn(C)
+        cs, ss = torch.zeros(seqs, 3, C, **f32), torch.zeros(seqs, C, **f32)
+        u = Y.conv_state(yx[:, C:], taps, bias, cs, seqs, rows // seqs, G)
+        wg, z = rn(G * 2 * n, 2 * n), torch.empty(rows, 2 * C, **f32)
+        add(tag + "conv", lambda yx=yx, cs=cs, seqs=seqs, rows=rows: Y.conv_state(yx[:, C:], taps, bias, cs, seqs,
+                                                                                 rows // seqs, G), rows * C * 6)
+        add(tag + "gates", lambda u=u, z=z: Y.grouped_gemm(seg(u, wg, z, groups=G, N_=2 * n, K=2 * n, x_col_stride=2 * n,
+                                                               out_col_stride=2 * n)),
+            rows * C * 12 + 8 * C * n, 8.0 * rows * C * n)
+        add(tag + "lru_scan", lambda u=u, z=z, yx=yx, ss=ss, seqs=seqs, rows=rows: Y.lru_scan(
+            u, z, bias, bias, bias, yx[:, :C], ss, seqs, rows // seqs, G, 8.0), rows * C * 16)
+        # ---- latent attention
+        d, gq, gc = rn(rows, Rq + R), rn(Rq), rn(R)
+        cache = rn(seqs, Sk, R)
+        pos = 0 if tag == "" else Sk - 1
+        add(tag + "latent_append", lambda d=d, cache=cache, seqs=seqs, rows=rows, pos=pos: Y.latent_norm_append(
+            d, gq, gc, cache, seqs, rows // seqs, pos, 1e-6), 4 * rows * (Rq + R))
+    ql, ukt, uv = rn(Bd, H * hd), rn(H * R, hd), rn(H * hd, R)
+    qa, ol, oo = torch.empty(Bd, H * R, **bf), rn(Bd, H * R), torch.empty(Bd, H * hd, **bf)
+    add("dec_absorb_q", lambda: Y.grouped_gemm(seg(ql, ukt, qa, groups=H, N_=R, K=hd, x_col_stride=hd, out_col_stride=R)),
+        2 * (H * R * hd + Bd * H * (hd + R)))
+    add("dec_absorb_v", lambda: Y.grouped_gemm(seg(ol, uv, oo, groups=H, N_=hd, K=R, x_col_stride=R, out_col_stride=hd)),
+        2 * (H * R * hd + Bd * H * (hd + R)))
+    splits, wsn = Y.latent_attn_plan(Bd, H, R, Sk, False)
+    ws = torch.empty(max(1, wsn), **f32)
+    add("dec_latent_attn", lambda: Y.latent_attn(ol, cache, Bd, 1, H, Sk - 1, 0.05, splits=splits, ws=ws),
+        2 * Bd * (Sk * R + 2 * H * R))
+    kc, vc, od = rn(Bd, Sk, 4 * hd), rn(Bd, Sk, 4 * hd), torch.empty(Bd, H * hd, **bf)
+    add("like_dec_attn", lambda: Dk.attn_decode(ql, kc, vc, Bd, 1, Sk, H, 4, hd, Sk - 1, out=od), 4 * Bd * Sk * 4 * hd)
+    qkv = rn(M, (H + 8) * hd)
+    kp, vp = rn(B, S, 4 * hd), rn(B, S, 4 * hd)
+    add("like_rope_append", lambda: Dk.rope_kv_append(qkv, kp, vp, B, S, H, 4, hd, 0), 4 * M * (H + 8) * hd)
+    hh, hw, hl = rn(Bd, D), rn(V, D), torch.empty(Bd, V, **f32)
+    add("dec_head", lambda: Y.grouped_gemm(seg(hh, hw, hl, groups=1, N_=V, K=D)), 2 * V * D + 4 * Bd * V)
+    gemm("like_dec_gate_up", Bd, 2 * 5464 // 8 * 8, D)
+    gemm("like_dec_down", Bd, D, 5464 // 8 * 8)
+    gemm("like_dec_qkv", Bd, (H + 8) * hd, D)
+    gemm("like_dec_head", Bd, V, D)
+    gemm("dec_dq_dkv", Bd, Rq + R, D)
     return cases
 
 

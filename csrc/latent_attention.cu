@@ -10,7 +10,7 @@
 //                        tensor-core fragments (heads are the 16 rows), which the 2 * 16 multiply-adds per cached byte
 //                        pair need: CUDA cores could not keep up with HBM.  Scores, maxima, exponentials and sums are
 //                        fp32, and the weights enter the second product as a high and a low bf16 part (16 mantissa bits).
-//                        The last CTA of a query folds the key slices.
+//   latent_attn_merge    folds the key slices of a query
 //   latent_attn_simt     any R and dtype (the fp32 path): one warp streams keys for one head
 #include <cuda_bf16.h>
 
@@ -34,28 +34,46 @@ struct LatentAppendParams {
   float eps;
 };
 
-// One warp per (token, projection).
-template <typename T>
+// One warp per (token, projection); V consecutive features per lane and load, the first kKeep loads stay in registers.
+template <typename T, int V>
 __global__ void __launch_bounds__(128) latent_norm_append_kernel(const LatentAppendParams p) {
+  constexpr int kKeep = V == 8 ? 3 : 4;
   const int wid = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int row = wid >> 1, which = wid & 1;
+  const int n = which ? p.R : p.Rq;
+  const T* g = static_cast<const T*>(which ? p.gc : p.gq);
   pdl_wait();
   pdl_launch_dependents();
-  const int row = wid >> 1, which = wid & 1;
   if (row >= p.B * p.S) return;
-  const int n = which ? p.R : p.Rq;
+  const int pos0 = p.pos_ptr ? *p.pos_ptr : p.pos;
   const T* src = static_cast<const T*>(p.d) + (long long)row * p.ldd + (which ? p.Rq : 0);
-  const T* g = static_cast<const T*>(which ? p.gc : p.gq);
-  float ss = 0.0f;
-  for (int i = lane; i < n; i += 32) {
-    const float v = to_f32(src[i]);
-    ss = fmaf(v, v, ss);
+  auto load = [&](const T* q, float (&o)[V]) {
+    if constexpr (V == 8) Vec8<T>::load(q, o);
+    else o[0] = to_f32(q[0]);
+  };
+  float v[kKeep][V], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (i * 32 + lane) * V;
+#pragma unroll
+    for (int k = 0; k < V; ++k) v[i][k] = 0.0f;
+    if (c < n) load(src + c, v[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i)
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+  for (int c = (kKeep * 32 + lane) * V; c < n; c += 32 * V) {
+    float t[V];
+    load(src + c, t);
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(t[k], t[k], ss);
   }
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + p.eps);
   T* dst;
   T* dst2 = nullptr;
   if (which) {
-    const int b = row / p.S, s = row % p.S;
-    const int at = (p.pos_ptr ? *p.pos_ptr : p.pos) + s;
+    const int b = row / p.S, at = pos0 + row % p.S;
     if (at < 0 || at >= p.cap) {
       if (lane == 0) report_error(kBadArgument);
       return;
@@ -65,10 +83,28 @@ __global__ void __launch_bounds__(128) latent_norm_append_kernel(const LatentApp
   } else {
     dst = static_cast<T*>(p.cq) + (long long)row * p.Rq;
   }
-  for (int i = lane; i < n; i += 32) {
-    const T v = from_f32<T>(to_f32(src[i]) * inv * to_f32(g[i]));
-    dst[i] = v;
-    if (dst2) dst2[i] = v;
+  auto put = [&](int c, const float (&x)[V]) {
+    float w[V], o[V];
+    load(g + c, w);
+#pragma unroll
+    for (int k = 0; k < V; ++k) o[k] = x[k] * inv * w[k];
+    if constexpr (V == 8) {
+      Vec8<T>::store(dst + c, o);
+      if (dst2) Vec8<T>::store(dst2 + c, o);
+    } else {
+      dst[c] = from_f32<T>(o[0]);
+      if (dst2) dst2[c] = from_f32<T>(o[0]);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (i * 32 + lane) * V;
+    if (c < n) put(c, v[i]);
+  }
+  for (int c = (kKeep * 32 + lane) * V; c < n; c += 32 * V) {
+    float t[V];
+    load(src + c, t);
+    put(c, t);
   }
 }
 
@@ -81,8 +117,7 @@ struct LatentAttnParams {
   const int* pos_ptr;
   float scale;
   int splits;
-  float* ws;                // [B*S * ceil(H/16)][splits][16][R + 2]
-  int* counters;            // [B*S * ceil(H/16)], zero between launches
+  float* ws;                // [B*S][H][splits][R + 4]: sums, then maximum and weight sum
 };
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -90,18 +125,17 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                : "r"(addr));
 }
-__device__ __forceinline__ void ldmatrix_x2(uint32_t (&r)[2], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
 }
-__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t (&r)[2], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
+__device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
       "{%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void cp_async_16(uint32_t dst, const void* src, bool valid) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
@@ -112,27 +146,27 @@ __device__ __forceinline__ void cp_async_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
-constexpr int kLaKeys = 64;       // keys per tile; each of the 4 warps scores 16 of them
-constexpr int kLaThreads = 128;
+constexpr int kLaKeys = 32;       // keys per tile: four 8-key column tiles, each scored by two warps (half of R each)
+constexpr int kLaThreads = 256;
+constexpr int kLaPs = kLaKeys + 4;
 
 __host__ __device__ inline int la_row_bytes(int R) { return R * 2 + 16; }   // padded: conflict-free ldmatrix rows
 __host__ __device__ inline int la_smem_bytes(int R) {
-  return (16 + 2 * kLaKeys) * la_row_bytes(R) + (16 * (kLaKeys + 4) + 16 * 3 + 4) * 4;
+  return (16 + 2 * kLaKeys) * la_row_bytes(R) + (2 * 16 * kLaPs + 16 * 3) * 4;
 }
 
-// MAXNT: 8-column tiles of the R output columns a warp can hold (R / 32 <= MAXNT).
-template <int MAXNT>
+// MAXP: pairs of 8-column output tiles a warp holds (R / 16 pairs over 8 warps).
+template <int MAXP>
 __global__ void __launch_bounds__(kLaThreads)
 latent_attn_mma_kernel(const LatentAttnParams p) {
   extern __shared__ __align__(16) uint8_t smem[];
   const int R = p.R, rb = la_row_bytes(R);
   uint8_t* qs = smem;
   uint8_t* cs = smem + 16 * rb;
-  float* ps = reinterpret_cast<float*>(cs + 2 * kLaKeys * rb);   // [16][kLaKeys + 4] scores, then weights
-  float* m_s = ps + 16 * (kLaKeys + 4);                          // [16] running maximum
+  float* ps = reinterpret_cast<float*>(cs + 2 * kLaKeys * rb);   // [2][16][kLaPs]: score halves; plane 0 then the weights
+  float* m_s = ps + 2 * 16 * kLaPs;                              // [16] running maximum
   float* l_s = m_s + 16;                                         // [16] running sum
   float* al_s = l_s + 16;                                        // [16] rescale of this tile
-  int* flag_s = reinterpret_cast<int*>(al_s + 16);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, hg = blockIdx.y, row = blockIdx.z;
@@ -144,22 +178,30 @@ latent_attn_mma_kernel(const LatentAttnParams p) {
   const int per = (n_tiles + p.splits - 1) / p.splits;
   const int t0 = split * per, t1 = min(n_tiles, t0 + per);
   const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache) + (long long)b * p.cap * R;
-  const int vec_per_row = R / 8;
+  const int vpr = R / 8;                                         // 16-byte pieces of a row
+  const int key_a = threadIdx.x / vpr, v_a = threadIdx.x % vpr;  // this thread's first piece of a tile ...
+  const int key_d = kLaThreads / vpr, v_d = kLaThreads % vpr;    // ... and the step to the next
 
   auto load_tile = [&](int t, int stage) {
-    uint8_t* dst = cs + stage * kLaKeys * rb;
-    for (int i = threadIdx.x; i < kLaKeys * vec_per_row; i += kLaThreads) {
-      const int key = i / vec_per_row, v = i % vec_per_row;
+    const uint32_t dst = smem_u32(cs + stage * kLaKeys * rb);
+    int key = key_a, v = v_a;
+    while (key < kLaKeys) {
       const int j = t * kLaKeys + key;
       const bool ok = j <= last;
-      cp_async_16(smem_u32(dst + key * rb + v * 16), cache + (long long)(ok ? j : last) * R + v * 8, ok);
+      cp_async_16(dst + key * rb + v * 16, cache + (long long)(ok ? j : last) * R + v * 8, ok);
+      key += key_d;
+      v += v_d;
+      if (v >= vpr) {
+        v -= vpr;
+        ++key;
+      }
     }
   };
   if (t0 < t1) load_tile(t0, 0);
   cp_async_commit();
   // the 16 heads' queries (rows past H are zero)
-  for (int i = threadIdx.x; i < 16 * vec_per_row; i += kLaThreads) {
-    const int hh = i / vec_per_row, v = i % vec_per_row;
+  for (int i = threadIdx.x; i < 16 * vpr; i += kLaThreads) {
+    const int hh = i / vpr, v = i % vpr;
     const int h = hg * 16 + hh;
     uint4 u = make_uint4(0, 0, 0, 0);
     if (h < p.H)
@@ -170,13 +212,16 @@ latent_attn_mma_kernel(const LatentAttnParams p) {
     m_s[threadIdx.x] = -INFINITY;
     l_s[threadIdx.x] = 0.0f;
   }
-  float acc[MAXNT][4];
+  float acc[MAXP][8];
 #pragma unroll
-  for (int n = 0; n < MAXNT; ++n)
+  for (int n = 0; n < MAXP; ++n)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) acc[n][i] = 0.0f;
-  const int nt = R / 32;                 // this warp's output columns: [warp * 8 * nt, + 8 * nt)
+    for (int i = 0; i < 8; ++i) acc[n][i] = 0.0f;
+  const int pairs = R / 16;              // this warp's output columns: 16-column pairs warp, warp + 8, ...
   const float sl2 = p.scale * 1.4426950408889634f;
+  const int nt = warp & 3, half = warp >> 2;      // scores: 8 keys, half of the features (R / 32 steps of 16)
+  const uint32_t q_addr = smem_u32(qs) + (lane & 15) * rb + (lane >> 4) * 16 + half * R;
+  const uint32_t k_off = (nt * 8 + (lane & 7)) * rb + (lane >> 3) * 16 + half * R;
 
   for (int t = t0; t < t1; ++t) {
     const int stage = (t - t0) & 1;
@@ -184,59 +229,59 @@ latent_attn_mma_kernel(const LatentAttnParams p) {
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    const uint8_t* ct = cs + stage * kLaKeys * rb;
-    // ---- scores of 16 heads x 16 keys
-    float s0[4] = {0, 0, 0, 0}, s1[4] = {0, 0, 0, 0};
-    const uint32_t qa = smem_u32(qs + (lane & 15) * rb + (lane >> 4) * 16);
-    const uint32_t kb = smem_u32(ct + (warp * 16 + (lane & 7)) * rb + ((lane >> 3) & 1) * 16);
-    for (int k = 0; k < R / 16; ++k) {
-      uint32_t a[4], b0[2], b1[2];
-      ldmatrix_x4(a, qa + k * 32);
-      ldmatrix_x2(b0, kb + k * 32);
-      ldmatrix_x2(b1, kb + 8 * rb + k * 32);
-      mma_bf16_16816(s0, a, b0);
-      mma_bf16_16816(s1, a, b1);
+    const uint32_t ct = smem_u32(cs + stage * kLaKeys * rb);
+    // ---- scores of 16 heads x 8 keys over half of R; four accumulators keep four products in flight
+    float s[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) s[i][k] = 0.0f;
+    const uint32_t kb = ct + k_off;
+    int k = 0;
+    for (; k + 4 <= R / 32; k += 4) {
+      uint32_t a[4][4], bb[2][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) ldmatrix_x4(a[i], q_addr + (k + i) * 32);
+      ldmatrix_x4(bb[0], kb + k * 32);
+      ldmatrix_x4(bb[1], kb + (k + 2) * 32);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) mma_bf16_16816(s[i], a[i], bb[i >> 1][(i & 1) * 2], bb[i >> 1][(i & 1) * 2 + 1]);
+    }
+    for (; k < R / 32; ++k) {            // (the upper half of the loaded key fragment belongs to the next step)
+      uint32_t a[4], bb[4];
+      ldmatrix_x4(a, q_addr + k * 32);
+      ldmatrix_x4(bb, kb + k * 32);
+      mma_bf16_16816(s[0], a, bb[0], bb[1]);
     }
     {
-      const int r0 = lane >> 2, c0 = warp * 16 + (lane & 3) * 2;
-      const int j0 = t * kLaKeys + c0;
-      float* pr0 = ps + r0 * (kLaKeys + 4);
-      float* pr1 = ps + (r0 + 8) * (kLaKeys + 4);
-      pr0[c0] = j0 <= last ? s0[0] * sl2 : -INFINITY;
-      pr0[c0 + 1] = j0 + 1 <= last ? s0[1] * sl2 : -INFINITY;
-      pr1[c0] = j0 <= last ? s0[2] * sl2 : -INFINITY;
-      pr1[c0 + 1] = j0 + 1 <= last ? s0[3] * sl2 : -INFINITY;
-      pr0[c0 + 8] = j0 + 8 <= last ? s1[0] * sl2 : -INFINITY;
-      pr0[c0 + 9] = j0 + 9 <= last ? s1[1] * sl2 : -INFINITY;
-      pr1[c0 + 8] = j0 + 8 <= last ? s1[2] * sl2 : -INFINITY;
-      pr1[c0 + 9] = j0 + 9 <= last ? s1[3] * sl2 : -INFINITY;
+      const int r0 = lane >> 2, c0 = nt * 8 + (lane & 3) * 2;
+      float* pr = ps + half * 16 * kLaPs + r0 * kLaPs + c0;
+      *reinterpret_cast<float2*>(pr) =
+          make_float2((s[0][0] + s[1][0]) + (s[2][0] + s[3][0]), (s[0][1] + s[1][1]) + (s[2][1] + s[3][1]));
+      *reinterpret_cast<float2*>(pr + 8 * kLaPs) =
+          make_float2((s[0][2] + s[1][2]) + (s[2][2] + s[3][2]), (s[0][3] + s[1][3]) + (s[2][3] + s[3][3]));
     }
     __syncthreads();
-    // ---- softmax: 8 threads per head, 8 keys each (a head's 8 threads are neighbours in one warp)
+    // ---- softmax: 16 threads per head, 2 keys each (a head's threads are neighbours in one warp)
     {
-      const int hh = threadIdx.x >> 3, part = threadIdx.x & 7;
-      float* pr = ps + hh * (kLaKeys + 4) + part * 8;
-      float v[8], mx = -INFINITY;
+      const int hh = threadIdx.x >> 4, c0 = (threadIdx.x & 15) * 2;
+      float* pr = ps + hh * kLaPs + c0;
+      const float2 x = *reinterpret_cast<const float2*>(pr);
+      const float2 y = *reinterpret_cast<const float2*>(pr + 16 * kLaPs);
+      const int j = t * kLaKeys + c0;
+      const float v0 = j <= last ? (x.x + y.x) * sl2 : -INFINITY;
+      const float v1 = j + 1 <= last ? (x.y + y.y) * sl2 : -INFINITY;
+      float mx = fmaxf(v0, v1);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        v[i] = pr[i];
-        mx = fmaxf(mx, v[i]);
-      }
-#pragma unroll
-      for (int o = 1; o < 8; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      for (int o = 1; o < 16; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_old = m_s[hh];
       const float m_new = fmaxf(m_old, mx);       // finite: every tile in range has a visible key
-      float sum = 0.0f;
+      const float w0 = exp2f(v0 - m_new), w1 = exp2f(v1 - m_new);
+      *reinterpret_cast<float2*>(pr) = make_float2(w0, w1);
+      float sum = w0 + w1;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        v[i] = exp2f(v[i] - m_new);
-        pr[i] = v[i];
-        sum += v[i];
-      }
-#pragma unroll
-      for (int o = 1; o < 8; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      __syncwarp();
-      if (part == 0) {
+      for (int o = 1; o < 16; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      if ((threadIdx.x & 15) == 0) {              // (the shuffles above order every lane's read of m_s before this)
         const float al = exp2f(m_old - m_new);
         al_s[hh] = al;
         m_s[hh] = m_new;
@@ -248,30 +293,38 @@ latent_attn_mma_kernel(const LatentAttnParams p) {
     {
       const int r0 = lane >> 2;
       const float al0 = al_s[r0], al1 = al_s[r0 + 8];
+      if (__any_sync(0xffffffffu, al0 != 1.0f || al1 != 1.0f)) {
 #pragma unroll
-      for (int n = 0; n < MAXNT; ++n) {
-        acc[n][0] *= al0; acc[n][1] *= al0;
-        acc[n][2] *= al1; acc[n][3] *= al1;
+        for (int n = 0; n < MAXP; ++n) {
+          acc[n][0] *= al0; acc[n][1] *= al0; acc[n][4] *= al0; acc[n][5] *= al0;
+          acc[n][2] *= al1; acc[n][3] *= al1; acc[n][6] *= al1; acc[n][7] *= al1;
+        }
       }
 #pragma unroll
-      for (int k = 0; k < kLaKeys / 16; ++k) {
+      for (int kk = 0; kk < kLaKeys / 16; ++kk) {
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {     // fragment register i: row + 8 * (i & 1), keys + 8 * (i >> 1)
-          const float2 w = *reinterpret_cast<const float2*>(ps + (r0 + 8 * (i & 1)) * (kLaKeys + 4) + k * 16 +
-                                                            8 * (i >> 1) + (lane & 3) * 2);
+          const float2 w = *reinterpret_cast<const float2*>(ps + (r0 + 8 * (i & 1)) * kLaPs + kk * 16 + 8 * (i >> 1) +
+                                                            (lane & 3) * 2);
           hi[i] = pack_bf16x2(w.x, w.y);
           const float2 h = unpack_bf16x2(hi[i]);
           lo[i] = pack_bf16x2(w.x - h.x, w.y - h.y);
         }
-        const uint32_t vb = smem_u32(ct + (k * 16 + (lane & 15)) * rb + warp * 16 * nt);
+        // lanes 0-15: the 16 keys' first 8 columns, lanes 16-31: the next 8
+        const uint32_t vb = ct + (kk * 16 + (lane & 15)) * rb + (lane >> 4) * 16;
 #pragma unroll
-        for (int n = 0; n < MAXNT; ++n) {
-          if (n < nt) {
-            uint32_t bv[2];
-            ldmatrix_x2_trans(bv, vb + n * 16);
-            mma_bf16_16816(acc[n], hi, bv);
-            mma_bf16_16816(acc[n], lo, bv);
+        for (int n = 0; n < MAXP; ++n) {
+          const int pr = warp + n * 8;
+          if (pr < pairs) {
+            uint32_t bv[4];
+            ldmatrix_x4_trans(bv, vb + pr * 32);
+            float(&d0)[4] = *reinterpret_cast<float(*)[4]>(&acc[n][0]);
+            float(&d1)[4] = *reinterpret_cast<float(*)[4]>(&acc[n][4]);
+            mma_bf16_16816(d0, hi, bv[0], bv[1]);
+            mma_bf16_16816(d1, hi, bv[2], bv[3]);
+            mma_bf16_16816(d0, lo, bv[0], bv[1]);
+            mma_bf16_16816(d1, lo, bv[2], bv[3]);
           }
         }
       }
@@ -279,67 +332,76 @@ latent_attn_mma_kernel(const LatentAttnParams p) {
     __syncthreads();      // the tile and the weights may be overwritten
   }
   cp_async_wait<0>();
+  __syncthreads();
 
   const int r0 = lane >> 2;
-  const int group = row * gridDim.y + hg;
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.o) + (long long)row * p.H * R;
-  if (p.splits == 1) {
-    const float i0 = 1.0f / l_s[r0], i1 = 1.0f / l_s[r0 + 8];
-    const int h0 = hg * 16 + r0, h1 = h0 + 8;
 #pragma unroll
-    for (int n = 0; n < MAXNT; ++n) {
-      if (n < nt) {
-        const int c = (warp * nt + n) * 8 + (lane & 3) * 2;
-        if (h0 < p.H) *reinterpret_cast<uint32_t*>(out + (long long)h0 * R + c) = pack_bf16x2(acc[n][0] * i0, acc[n][1] * i0);
-        if (h1 < p.H) *reinterpret_cast<uint32_t*>(out + (long long)h1 * R + c) = pack_bf16x2(acc[n][2] * i1, acc[n][3] * i1);
+  for (int hr = 0; hr < 2; ++hr) {
+    const int hh = r0 + hr * 8, h = hg * 16 + hh;
+    if (h >= p.H) continue;
+    if (p.splits == 1) {
+      const float inv = 1.0f / l_s[hh];
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.o) + ((long long)row * p.H + h) * R;
+#pragma unroll
+      for (int n = 0; n < MAXP; ++n) {
+        const int pr = warp + n * 8;
+        if (pr >= pairs) continue;
+        const int c = pr * 16 + (lane & 3) * 2;
+        *reinterpret_cast<uint32_t*>(out + c) = pack_bf16x2(acc[n][hr * 2] * inv, acc[n][hr * 2 + 1] * inv);
+        *reinterpret_cast<uint32_t*>(out + c + 8) = pack_bf16x2(acc[n][4 + hr * 2] * inv, acc[n][4 + hr * 2 + 1] * inv);
+      }
+    } else {
+      float* mine = p.ws + (((long long)row * p.H + h) * p.splits + split) * (R + 4);
+#pragma unroll
+      for (int n = 0; n < MAXP; ++n) {
+        const int pr = warp + n * 8;
+        if (pr >= pairs) continue;
+        const int c = pr * 16 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(mine + c) = make_float2(acc[n][hr * 2], acc[n][hr * 2 + 1]);
+        *reinterpret_cast<float2*>(mine + c + 8) = make_float2(acc[n][4 + hr * 2], acc[n][4 + hr * 2 + 1]);
+      }
+      if (warp == 0 && (lane & 3) == 0) {
+        mine[R] = m_s[hh];
+        mine[R + 1] = l_s[hh];
       }
     }
-    return;
   }
-  // ---- partials, and the fold by the CTA that arrives last
-  const int st = R + 2;
-  float* mine = p.ws + ((long long)group * p.splits + split) * 16 * st;
-#pragma unroll
-  for (int n = 0; n < MAXNT; ++n) {
-    if (n < nt) {
-      const int c = (warp * nt + n) * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(mine + r0 * st + c) = make_float2(acc[n][0], acc[n][1]);
-      *reinterpret_cast<float2*>(mine + (r0 + 8) * st + c) = make_float2(acc[n][2], acc[n][3]);
-    }
+}
+
+// One CTA per (query, head): o' = sum over slices of 2^(m_s - m) x_s / sum of the rescaled weight sums.
+__global__ void __launch_bounds__(128) latent_attn_merge_kernel(const LatentAttnParams p) {
+  __shared__ float wt[64];
+  __shared__ float inv_s;
+  const int R = p.R, st = R + 4;
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long rh = blockIdx.x;
+  const float* base = p.ws + rh * p.splits * st;
+  if (threadIdx.x < 32) {
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
+    const int s0 = threadIdx.x, s1 = threadIdx.x + 32;
+    if (s0 < p.splits) { m0 = __ldcg(base + s0 * st + R); l0 = __ldcg(base + s0 * st + R + 1); }
+    if (s1 < p.splits) { m1 = __ldcg(base + s1 * st + R); l1 = __ldcg(base + s1 * st + R + 1); }
+    const float m = warp_max(fmaxf(m0, m1));
+    const float w0 = exp2f(m0 - m), w1 = exp2f(m1 - m);      // an empty slice has maximum -inf: weight 0
+    const float l = warp_sum(l0 * w0 + l1 * w1);
+    wt[s0] = w0;
+    wt[s1] = w1;
+    if (threadIdx.x == 0) inv_s = 1.0f / l;
   }
   __syncthreads();
-  if (threadIdx.x < 16) {
-    mine[threadIdx.x * st + R] = m_s[threadIdx.x];
-    mine[threadIdx.x * st + R + 1] = l_s[threadIdx.x];
-  }
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    const int old = atomicAdd(&p.counters[group], 1);
-    *flag_s = old == p.splits - 1;
-    if (old == p.splits - 1) p.counters[group] = 0;
-  }
-  __syncthreads();
-  if (!*flag_s) return;
-  __threadfence();
-  const float* base = p.ws + (long long)group * p.splits * 16 * st;
-  for (int i = threadIdx.x; i < 16 * (R / 2); i += kLaThreads) {
-    const int hh = i / (R / 2), c = (i % (R / 2)) * 2;
-    const int h = hg * 16 + hh;
-    if (h >= p.H) continue;
-    float m = -INFINITY;
-    for (int s = 0; s < p.splits; ++s) m = fmaxf(m, __ldcg(base + (s * 16 + hh) * st + R));
-    float l = 0.0f, x = 0.0f, y = 0.0f;
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.o) + rh * R;
+  for (int c = threadIdx.x * 4; c < R; c += 512) {
+    float x[4] = {0, 0, 0, 0};
+#pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
-      const float* q = base + (s * 16 + hh) * st;
-      const float w = exp2f(__ldcg(q + R) - m);       // an empty slice has maximum -inf: weight 0
-      const float2 v = __ldcg(reinterpret_cast<const float2*>(q + c));
-      l = fmaf(__ldcg(q + R + 1), w, l);
-      x = fmaf(v.x, w, x);
-      y = fmaf(v.y, w, y);
+      const float4 v = __ldcg(reinterpret_cast<const float4*>(base + s * st + c));
+      const float w = wt[s];
+      x[0] = fmaf(v.x, w, x[0]); x[1] = fmaf(v.y, w, x[1]);
+      x[2] = fmaf(v.z, w, x[2]); x[3] = fmaf(v.w, w, x[3]);
     }
-    const float inv = 1.0f / l;
-    *reinterpret_cast<uint32_t*>(out + (long long)h * R + c) = pack_bf16x2(x * inv, y * inv);
+    const float inv = inv_s;
+    *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16x2(x[0] * inv, x[1] * inv), pack_bf16x2(x[2] * inv, x[3] * inv));
   }
 }
 
@@ -403,16 +465,18 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const LatentAttnP
   }
 }
 
-template <int MAXNT>
+template <int MAXP>
 static int launch_latent_mma(const LatentAttnParams& p, dim3 grid, cudaStream_t st) {
-  auto kern = latent_attn_mma_kernel<MAXNT>;
+  auto kern = latent_attn_mma_kernel<MAXP>;
   const int bytes = la_smem_bytes(p.R);
   static int configured = 0;
   if (configured < bytes) {
     DPTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
     configured = bytes;
   }
-  return counted(1, (int)launch_k(kern, grid, dim3(kLaThreads), (size_t)bytes, st, p));
+  const int rc = counted(1, (int)launch_k(kern, grid, dim3(kLaThreads), (size_t)bytes, st, p));
+  if (rc || p.splits == 1) return rc;
+  return counted(1, (int)launch_k(latent_attn_merge_kernel, dim3((unsigned)(p.B * p.S * p.H)), dim3(128), (size_t)0, st, p));
 }
 template <typename T>
 static int launch_latent_simt(const LatentAttnParams& p, cudaStream_t st) {
@@ -431,11 +495,11 @@ using namespace dptb;
 
 struct DptbLatentArgs {
   const void* d; const void* gq; const void* gc; void* cq; void* c_new;      // append
-  const void* q; void* o; float* ws; int* counters;                          // attention
+  const void* q; void* o; float* ws;                                         // attention
   void* cache;
   const int* pos_ptr;
   long long ldd, ws_floats;
-  int B, S, H, Rq, R, cap, pos, splits, num_counters, f32, force_simt;
+  int B, S, H, Rq, R, cap, pos, splits, f32, force_simt;
   float eps, scale;
 };
 
@@ -448,25 +512,28 @@ extern "C" int dptb_latent_norm_append(const DptbLatentArgs* a, void* stream_v) 
   p.d = a->d; p.ldd = a->ldd; p.gq = a->gq; p.gc = a->gc; p.cq = a->cq; p.cache = a->cache; p.c_new = a->c_new;
   p.B = a->B; p.S = a->S; p.Rq = a->Rq; p.R = a->R; p.cap = a->cap; p.pos = a->pos; p.pos_ptr = a->pos_ptr; p.eps = a->eps;
   const dim3 grid((2 * a->B * a->S + 3) / 4);
-  return counted(1, (int)(a->f32 ? launch_k(latent_norm_append_kernel<float>, grid, dim3(128), (size_t)0, st, p)
-                                 : launch_k(latent_norm_append_kernel<__nv_bfloat16>, grid, dim3(128), (size_t)0, st, p)));
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = a->Rq % 8 == 0 && a->R % 8 == 0 && a->ldd % 8 == 0 && al16(a->d) && al16(a->gq) && al16(a->gc) &&
+                   al16(a->cq) && al16(a->cache) && (!a->c_new || al16(a->c_new));
+  auto kern = a->f32 ? (vec ? latent_norm_append_kernel<float, 8> : latent_norm_append_kernel<float, 1>)
+                     : (vec ? latent_norm_append_kernel<__nv_bfloat16, 8> : latent_norm_append_kernel<__nv_bfloat16, 1>);
+  return counted(1, (int)launch_k(kern, grid, dim3(128), (size_t)0, st, p));
 }
 
 static bool latent_mma_ok(int R, int f32) { return !f32 && R % 32 == 0 && R <= 512; }
 
-// Key slices per query: enough CTAs to fill the SMs, at least two key tiles each at the largest context.
+// Key slices per query: enough CTAs to fill the SMs, at least four key tiles each at the largest context.
 extern "C" int dptb_latent_attn_splits(int rows, int H, int R, int max_keys, int f32) {
   if (!latent_mma_ok(R, f32)) return 1;
   const int groups = rows * ((H + 15) / 16);
-  const int per_sm = la_smem_bytes(R) <= 100 * 1024 ? 2 : 1;
-  int s = (sm_count() * per_sm) / (groups > 0 ? groups : 1);
-  const int by_keys = (max_keys + 2 * kLaKeys - 1) / (2 * kLaKeys);
+  int s = (sm_count() * 2) / (groups > 0 ? groups : 1);
+  const int by_keys = (max_keys + 4 * kLaKeys - 1) / (4 * kLaKeys);
   if (s > by_keys) s = by_keys;
   if (s > 64) s = 64;
   return s < 1 ? 1 : s;
 }
 extern "C" long long dptb_latent_attn_ws_floats(int rows, int H, int R, int splits) {
-  return splits <= 1 ? 0 : (long long)rows * ((H + 15) / 16) * splits * 16 * (R + 2);
+  return splits <= 1 ? 0 : (long long)rows * H * splits * (R + 4);
 }
 
 extern "C" int dptb_latent_attn(const DptbLatentArgs* a, void* stream_v) {
@@ -478,20 +545,18 @@ extern "C" int dptb_latent_attn(const DptbLatentArgs* a, void* stream_v) {
   LatentAttnParams p;
   p.q = a->q; p.cache = a->cache; p.o = a->o;
   p.B = a->B; p.S = a->S; p.H = a->H; p.R = a->R; p.cap = a->cap; p.pos = a->pos; p.pos_ptr = a->pos_ptr;
-  p.scale = a->scale; p.splits = a->splits < 1 ? 1 : a->splits; p.ws = a->ws; p.counters = a->counters;
+  p.scale = a->scale; p.splits = a->splits < 1 ? 1 : a->splits; p.ws = a->ws;
   if (rows > 65535) return kErrTooLarge;
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   if (!a->force_simt && latent_mma_ok(a->R, a->f32) && al16(a->q) && al16(a->cache) && al16(a->o)) {
     const int hg = (a->H + 15) / 16;
-    if (p.splits > 1 && (!a->ws || !a->counters || rows * hg > a->num_counters ||
-                         dptb_latent_attn_ws_floats(rows, a->H, a->R, p.splits) > a->ws_floats))
+    if (p.splits > 64 || (p.splits > 1 && (!a->ws || !al16(a->ws) ||
+                                           dptb_latent_attn_ws_floats(rows, a->H, a->R, p.splits) > a->ws_floats)))
       return kErrTooLarge;
     const dim3 grid(p.splits, hg, rows);
-    const int nt = a->R / 32;
-    if (nt <= 2) return launch_latent_mma<2>(p, grid, st);
-    if (nt <= 4) return launch_latent_mma<4>(p, grid, st);
-    if (nt <= 8) return launch_latent_mma<8>(p, grid, st);
-    return launch_latent_mma<16>(p, grid, st);
+    if (a->R <= 128) return launch_latent_mma<1>(p, grid, st);
+    if (a->R <= 256) return launch_latent_mma<2>(p, grid, st);
+    return launch_latent_mma<4>(p, grid, st);
   }
   return a->f32 ? launch_latent_simt<float>(p, st) : launch_latent_simt<__nv_bfloat16>(p, st);
 }

@@ -58,49 +58,82 @@ __device__ __forceinline__ void choose_top(float* sel, int E, int top, int lane,
   if (lane < top) w[lane] = mine / sum;
 }
 
+constexpr int kRouterThreads = 512;
+
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kRouterThreads)
 moe_router_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ router, int D, int E, int top, int* idx,
                   float* w, int* count) {
-  extern __shared__ float sm[];       // [D] the token, [E] logits
+  extern __shared__ __align__(16) float sm[];       // [D] the token, [E] logits
   float* logit = sm + D;
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  constexpr int kWarps = kRouterThreads / 32, kAtOnce = 4;      // a warp works on four experts at a time
   pdl_wait();
   pdl_launch_dependents();
-  for (int i = threadIdx.x; i < D; i += 256) sm[i] = to_f32(x[(long long)t * ldx + i]);
+  for (int i = threadIdx.x; i < D; i += kRouterThreads) sm[i] = to_f32(x[(long long)t * ldx + i]);
   __syncthreads();
-  for (int e = warp; e < E; e += 8) {
-    const T* r = router + (long long)e * D;
-    float acc = 0.0f;
-    if (D % 8 == 0) {
-      for (int i = lane * 8; i < D; i += 256) {
-        float v[8];
-        Vec8<T>::load(r + i, v);
+  for (int e0 = warp; e0 < E; e0 += kWarps * kAtOnce) {
+    float acc[kAtOnce];
+    const T* r[kAtOnce];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) acc = fmaf(v[k], sm[i + k], acc);
+    for (int q = 0; q < kAtOnce; ++q) {
+      acc[q] = 0.0f;
+      r[q] = router + (long long)min(e0 + q * kWarps, E - 1) * D;
+    }
+    if (D % 8 == 0) {
+#pragma unroll 2
+      for (int i = lane * 8; i < D; i += 256) {
+        Raw8<T> raw[kAtOnce];
+#pragma unroll
+        for (int q = 0; q < kAtOnce; ++q) raw[q].load(r[q] + i);
+        float xv[8];
+        Vec8<float>::load(sm + i, xv);
+#pragma unroll
+        for (int q = 0; q < kAtOnce; ++q) {
+          float v[8];
+          raw[q].unpack(v);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) acc[q] = fmaf(v[k], xv[k], acc[q]);
+        }
       }
     } else {
-      for (int i = lane; i < D; i += 32) acc = fmaf(to_f32(r[i]), sm[i], acc);
+      for (int i = lane; i < D; i += 32)
+#pragma unroll
+        for (int q = 0; q < kAtOnce; ++q) acc[q] = fmaf(to_f32(r[q][i]), sm[i], acc[q]);
     }
-    acc = warp_sum(acc);
-    if (lane == 0) logit[e] = acc;
+#pragma unroll
+    for (int q = 0; q < kAtOnce; ++q) {
+      const float z = warp_sum(acc[q]);
+      if (lane == 0 && e0 + q * kWarps < E) logit[e0 + q * kWarps] = z;
+    }
   }
   __syncthreads();
   if (warp == 0) choose_top(logit, E, top, lane, idx + (long long)t * top, w + (long long)t * top, count);
 }
 
+constexpr int kTopkTokens = 32;       // per CTA, so that a count costs one global atomic per CTA and expert
+
 __global__ void __launch_bounds__(256)
 moe_topk_kernel(const float* __restrict__ logits, long long ld, int T_, int E, int top, int* idx, float* w, int* count) {
-  extern __shared__ float sm[];       // [8][E]
+  extern __shared__ __align__(16) float sm[];       // [8][E] logits, [E] counts
+  int* hist = reinterpret_cast<int*>(sm + 8 * E);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int t = blockIdx.x * 8 + warp;
+  for (int e = threadIdx.x; e < E; e += 256) hist[e] = 0;
   pdl_wait();
   pdl_launch_dependents();
-  if (t >= T_) return;
+  __syncthreads();
   float* sel = sm + warp * E;
-  for (int e = lane; e < E; e += 32) sel[e] = logits[(long long)t * ld + e];
-  __syncwarp();
-  choose_top(sel, E, top, lane, idx + (long long)t * top, w + (long long)t * top, count);
+  for (int i = warp; i < kTopkTokens; i += 8) {
+    const long long t = (long long)blockIdx.x * kTopkTokens + i;
+    if (t >= T_) break;
+    for (int e = lane; e < E; e += 32) sel[e] = logits[t * ld + e];
+    __syncwarp();
+    choose_top(sel, E, top, lane, idx + t * top, w + t * top, hist);
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += 256)
+    if (hist[e]) atomicAdd(&count[e], hist[e]);
 }
 
 constexpr int kPlacePairs = 32;
@@ -183,16 +216,16 @@ extern "C" int dptb_moe_router(const DptbMoeArgs* a, void* stream_v) {
   if (a->T <= 0) return 0;
   if (a->E < 1 || a->E > kMoeMaxExperts || a->top < 1 || a->top > kMoeMaxTop || a->top > a->E || a->D < 1) return kErrBadShape;
   if (a->logits) {
-    return counted(1, (int)launch_k(moe_topk_kernel, dim3((a->T + 7) / 8), dim3(256), (size_t)8 * a->E * 4, st, a->logits,
+    return counted(1, (int)launch_k(moe_topk_kernel, dim3((a->T + kTopkTokens - 1) / kTopkTokens), dim3(256), (size_t)9 * a->E * 4, st, a->logits,
                                     a->ld_logits, a->T, a->E, a->top, a->idx, a->w, a->count));
   }
   const size_t bytes = (size_t)(a->D + a->E) * 4;
   if (bytes > 48 * 1024) return kErrTooLarge;
   if (a->D % 8 == 0 && (reinterpret_cast<uintptr_t>(a->router) & 15)) return kErrBadShape;
   if (a->f32)
-    return counted(1, (int)launch_k(moe_router_kernel<float>, dim3(a->T), dim3(256), bytes, st, (const float*)a->x, a->ldx,
+    return counted(1, (int)launch_k(moe_router_kernel<float>, dim3(a->T), dim3(kRouterThreads), bytes, st, (const float*)a->x, a->ldx,
                                     (const float*)a->router, a->D, a->E, a->top, a->idx, a->w, a->count));
-  return counted(1, (int)launch_k(moe_router_kernel<__nv_bfloat16>, dim3(a->T), dim3(256), bytes, st,
+  return counted(1, (int)launch_k(moe_router_kernel<__nv_bfloat16>, dim3(a->T), dim3(kRouterThreads), bytes, st,
                                   (const __nv_bfloat16*)a->x, a->ldx, (const __nv_bfloat16*)a->router, a->D, a->E, a->top,
                                   a->idx, a->w, a->count));
 }

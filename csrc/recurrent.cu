@@ -8,9 +8,10 @@
 //   conv_state_kernel   the convolution; its result leaves as a high and a low bf16 part side by side per block of
 //                       channels, so that the block-diagonal gate product (grouped tensor-core GEMM over [high | low]
 //                       against [W | W]) sees 16 mantissa bits; in fp32 it is one plain value
-//   lru_scan kernels    gates, decay and recurrence.  Up to one chunk of tokens: a single pass, one thread per channel.
-//                       Longer inputs: pass 1 leaves every chunk's total log decay and end state, pass 2 folds the
-//                       chunks before its own and runs the recurrence again from there.
+//   lru_scan kernels    gates, decay and recurrence, a thread per channel (or two).  Up to one chunk of tokens: a single
+//                       pass.  Longer inputs: pass 1 runs every chunk from a zero state and replaces the gate products
+//                       by the log decay since the chunk's start and that local state; pass 2 folds the ends of the
+//                       chunks before its own into the state it starts from and adds its decayed rest to every token.
 #include <cuda_bf16.h>
 
 #include "common/host.h"
@@ -94,9 +95,75 @@ __global__ void __launch_bounds__(128) conv_state_kernel(const ConvStateParams p
   put(t, acc);
 }
 
+// Eight channels per thread, runs of kConvRun rows, up to four taps, the window in registers.
+constexpr int kConvRun = 8;
+__global__ void __launch_bounds__(128) conv_state_vec_kernel(const ConvStateParams p) {
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
+  const int runs = (p.S + kConvRun - 1) / kConvRun;
+  const int b = blockIdx.x / runs, t0 = (blockIdx.x % runs) * kConvRun;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (c >= p.C) return;
+  const int K = p.K, hist = K - 1;
+  const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(p.x) + (long long)b * p.S * p.ldx + c;
+  const __nv_bfloat16* taps = static_cast<const __nv_bfloat16*>(p.taps) + (long long)c * K;
+  float w[4][8], win[4][8], bias[8];      // tap 3 is the current row's; win[3] the current row
+#pragma unroll
+  for (int k = 0; k < 4; ++k)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w[k][e] = k >= 4 - K ? __bfloat162float(taps[e * K + k - (4 - K)]) : 0.0f;
+  Vec8<__nv_bfloat16>::load(static_cast<const __nv_bfloat16*>(p.bias) + c, bias);
+  float* st = p.state + (long long)b * hist * p.C + c;
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {           // the three rows before t0
+    const int t = t0 - 3 + i, s = t + hist;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) win[i][e] = 0.0f;
+    if (t >= 0) Vec8<__nv_bfloat16>::load(x + (long long)t * p.ldx, win[i]);
+    else if (s >= 0) Vec8<float>::load(st + (long long)s * p.C, win[i]);
+  }
+  if (t0 == 0 && hist > 0) {              // the only thread that touches this sequence's state: read above, written here
+    for (int i = 0; i < hist; ++i) {
+      const int t = p.S - hist + i;
+      float v[8];
+      if (t >= 0) {
+        Vec8<__nv_bfloat16>::load(x + (long long)t * p.ldx, v);
+      } else {                            // fewer new rows than the state holds: the old state moves up
+        const int from = i + p.S - hist + 3;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = from == 0 ? win[0][e] : (from == 1 ? win[1][e] : win[2][e]);
+      }
+      Vec8<float>::store(st + (long long)i * p.C, v);
+    }
+  }
+  const int bw = p.C / p.blocks;
+  __nv_bfloat16* o = static_cast<__nv_bfloat16*>(p.u) + (long long)(c / bw) * 2 * bw + c % bw;
+  const int t1 = min(p.S, t0 + kConvRun);
+#pragma unroll
+  for (int i = 0; i < kConvRun; ++i) {
+    const int t = t0 + i;
+    if (t < t1) {
+      Vec8<__nv_bfloat16>::load(x + (long long)t * p.ldx, win[(i + 3) & 3]);
+      float hi[8], lo[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float acc = bias[e];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) acc = fmaf(w[k][e], win[(i + k) & 3][e], acc);
+        hi[e] = __bfloat162float(__float2bfloat16(acc));
+        lo[e] = acc - hi[e];
+      }
+      __nv_bfloat16* dst = o + ((long long)b * p.S + t) * 2 * p.C;
+      Vec8<__nv_bfloat16>::store(dst, hi);
+      Vec8<__nv_bfloat16>::store(dst + bw, lo);
+    }
+  }
+}
+
 struct LruParams {
   const void* u;            // as written by conv_state_kernel
-  const float* z;           // [B*S, blocks, 2, C / blocks] gate products without bias: recurrence gate, input gate
+  float* z;                 // [B*S, blocks, 2, C / blocks] gate products without bias: recurrence gate, input gate (pass 1
+                            // overwrites them)
   const void* br;           // [C]
   const void* bi;           // [C]
   const void* lam;          // [C]
@@ -109,17 +176,37 @@ struct LruParams {
   float c;
 };
 
-__device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
+// The math of one token.  The fp32 path calls the accurate functions; the bf16 path's inputs and outputs are rounded to
+// 8 bits, so the hardware exponential (relative error about 2^-21) is far below them.
+template <bool FAST>
+__device__ __forceinline__ float exp_f(float v) { return FAST ? __expf(v) : expf(v); }
+template <bool FAST>
+__device__ __forceinline__ float sigmoid_f(float v) {
+  return FAST ? __fdividef(1.0f, 1.0f + __expf(-v)) : 1.0f / (1.0f + expf(-v));
+}
+// e^v - 1 for v <= 0 with its relative precision next to 0: the Taylor polynomial of degree 7 up to 1/4
+template <bool FAST>
+__device__ __forceinline__ float expm1_neg_f(float v) {
+  if (!FAST) return expm1f(v);
+  const float t = v * fmaf(v, fmaf(v, fmaf(v, fmaf(v, fmaf(v, fmaf(v, 1.0f / 5040, 1.0f / 720), 1.0f / 120), 1.0f / 24),
+                                         1.0f / 6), 0.5f), 1.0f);
+  return v > -0.25f ? t : __expf(v) - 1.0f;
+}
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
+template <bool FAST>
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  // 1/2 (1 + tanh u) = sigmoid(2 u)
+  return FAST ? z * sigmoid_f<true>(2.0f * u) : 0.5f * z * (1.0f + tanhf(u));
 }
 
-template <typename T>
+// V neighbouring channels of one sequence.
+template <typename T, int V>
 struct LruChannel {
+  static constexpr bool FAST = sizeof(T) == 2;
   const T* u;
-  const float* z;
-  float br, bi, decay;      // decay = -c * softplus(lam)
+  float* z;
+  float br[V], bi[V], decay[V];      // decay = -c * softplus(lam)
   int bw, C;
   __device__ __forceinline__ LruChannel(const LruParams& p, int b, int ch) {
     bw = p.C / p.blocks;
@@ -127,83 +214,205 @@ struct LruChannel {
     const long long off = (long long)(ch / bw) * 2 * bw + ch % bw;
     const long long row0 = (long long)b * p.S;
     z = p.z + row0 * 2 * C + off;
-    u = static_cast<const T*>(p.u) + (sizeof(T) == 2 ? row0 * 2 * C + off : row0 * C + ch);
-    br = to_f32(static_cast<const T*>(p.br)[ch]);
-    bi = to_f32(static_cast<const T*>(p.bi)[ch]);
-    decay = -p.c * softplus_f(to_f32(static_cast<const T*>(p.lam)[ch]));
-  }
-  // Applies token t to S; returns its log decay.  With e = a - 1 = expm1(log a), which keeps its relative precision where
-  // a is next to 1:  1 - a^2 = -e (2 + e)  and  a S = S + e S, so long memories do not drift.
-  __device__ __forceinline__ float step(int t, float& S) const {
-    const float* zt = z + (long long)t * 2 * C;
-    float uv;
-    if constexpr (sizeof(T) == 2) {
-      const T* ut = u + (long long)t * 2 * C;
-      uv = to_f32(ut[0]) + to_f32(ut[bw]);
-    } else {
-      uv = to_f32(u[(long long)t * C]);
+    u = static_cast<const T*>(p.u) + (FAST ? row0 * 2 * C + off : row0 * C + ch);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      br[k] = to_f32(static_cast<const T*>(p.br)[ch + k]);
+      bi[k] = to_f32(static_cast<const T*>(p.bi)[ch + k]);
+      decay[k] = -p.c * softplus_f(to_f32(static_cast<const T*>(p.lam)[ch + k]));
     }
-    const float log_a = decay * sigmoid_f(zt[0] + br);
-    const float e = expm1f(log_a);
-    S += fmaf(e, S, sqrtf(-e * (2.0f + e)) * sigmoid_f(zt[bw] + bi) * uv);
-    return log_a;
+  }
+  template <typename U>
+  static __device__ __forceinline__ void load(const U* q, float (&o)[V]) {
+    if constexpr (V == 2 && sizeof(U) == 2) {
+      const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(q));
+      o[0] = f.x; o[1] = f.y;
+    } else if constexpr (V == 2) {
+      const float2 f = *reinterpret_cast<const float2*>(q);
+      o[0] = f.x; o[1] = f.y;
+    } else {
+      o[0] = to_f32(q[0]);
+    }
+  }
+  static __device__ __forceinline__ void store_f32(float* q, const float (&v)[V]) {
+    if constexpr (V == 2) *reinterpret_cast<float2*>(q) = make_float2(v[0], v[1]);
+    else q[0] = v[0];
+  }
+  // What token t brings; kept apart from the arithmetic so that several tokens' loads are in flight before any store.
+  struct In {
+    float zr[V], zi[V], u[V];
+  };
+  __device__ __forceinline__ void fetch(int t, In& in) const {
+    const float* zt = z + (long long)t * 2 * C;
+    load(zt, in.zr);
+    load(zt + bw, in.zi);
+    if constexpr (FAST) {
+      const T* ut = u + (long long)t * 2 * C;
+      float lo[V];
+      load(ut, in.u);
+      load(ut + bw, lo);
+#pragma unroll
+      for (int k = 0; k < V; ++k) in.u[k] += lo[k];
+    } else {
+      load(u + (long long)t * C, in.u);
+    }
+  }
+  // Applies a token to S; its log decay comes back in log_a.  With e = a - 1 = expm1(log a), which keeps its relative
+  // precision where a is next to 1:  1 - a^2 = -e (2 + e)  and  a S = S + e S, so long memories do not drift.
+  __device__ __forceinline__ void step(const In& in, float (&S)[V], float (&log_a)[V]) const {
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      log_a[k] = decay[k] * sigmoid_f<FAST>(in.zr[k] + br[k]);
+      const float e = expm1_neg_f<FAST>(log_a[k]);
+      S[k] += fmaf(e, S[k], sqrtf(-e * (2.0f + e)) * sigmoid_f<FAST>(in.zi[k] + bi[k]) * in.u[k]);
+    }
   }
 };
 
-// Pass 1: chunks 0 .. chunks-2; chunk 0 starts from the state and keeps a copy of it.
-template <typename T>
-__global__ void __launch_bounds__(128) lru_chunk_kernel(const LruParams p) {
-  const int ch = blockIdx.x * 128 + threadIdx.x, k = blockIdx.y, b = blockIdx.z;
-  pdl_wait();
-  pdl_launch_dependents();
-  if (ch >= p.C) return;
-  const LruChannel<T> lc(p, b, ch);
-  float* agg = p.agg + (long long)b * (p.chunks + 1) * 2 * p.C + ch;
-  float S = 0.0f, total = 0.0f;
-  if (k == 0) {
-    S = p.state[(long long)b * p.C + ch];
-    agg[(long long)p.chunks * 2 * p.C] = S;
+constexpr int kLruBatch = 4;      // tokens fetched at a time
+
+template <typename T, int V>
+__device__ __forceinline__ void lru_put(T* out, const float (&S)[V], const float (&y)[V]) {
+  float o[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) o[k] = S[k] * gelu_tanh_f<sizeof(T) == 2>(y[k]);
+  if constexpr (V == 2 && sizeof(T) == 2) {
+    *reinterpret_cast<uint32_t*>(out) = pack_bf16x2(o[0], o[1]);
+  } else {
+#pragma unroll
+    for (int k = 0; k < V; ++k) out[k] = from_f32<T>(o[k]);
   }
-  const int t0 = k * p.chunk, t1 = t0 + p.chunk;
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-    total += lc.step(t, S);
-  }
-  agg[(long long)k * 2 * p.C] = total;
-  agg[((long long)k * 2 + 1) * p.C] = S;
 }
 
-// Pass 2 (or the only pass when chunks == 1).
-template <typename T>
+// The whole recurrence in one pass (chunks == 1).
+template <typename T, int V>
 __global__ void __launch_bounds__(128) lru_scan_kernel(const LruParams p) {
-  const int ch = blockIdx.x * 128 + threadIdx.x, k = blockIdx.y, b = blockIdx.z;
+  const int ch = (blockIdx.x * 128 + threadIdx.x) * V, b = blockIdx.z;
   pdl_wait();
   pdl_launch_dependents();
   if (ch >= p.C) return;
-  const LruChannel<T> lc(p, b, ch);
-  float S;
-  if (p.chunks == 1) {
-    S = p.state[(long long)b * p.C + ch];
-  } else {
-    const float* agg = p.agg + (long long)b * (p.chunks + 1) * 2 * p.C + ch;
-    if (k == 0) {
-      S = agg[(long long)p.chunks * 2 * p.C];
-    } else {
-      S = agg[p.C];
-#pragma unroll 4
-      for (int j = 1; j < k; ++j)
-        S += fmaf(expm1f(agg[(long long)j * 2 * p.C]), S, agg[((long long)j * 2 + 1) * p.C]);
+  const LruChannel<T, V> lc(p, b, ch);
+  float* state = p.state + (long long)b * p.C + ch;
+  float S[V], la[V], y[kLruBatch][V];
+  LruChannel<T, V>::load(state, S);
+  const T* yp = static_cast<const T*>(p.y) + (long long)b * p.S * p.ldy + ch;
+  T* out = static_cast<T*>(p.out) + (long long)b * p.S * p.C + ch;
+  typename LruChannel<T, V>::In in[kLruBatch];
+  for (int t0 = 0; t0 < p.S; t0 += kLruBatch) {
+#pragma unroll
+    for (int i = 0; i < kLruBatch; ++i) {
+      if (t0 + i < p.S) {
+        lc.fetch(t0 + i, in[i]);
+        LruChannel<T, V>::load(yp + (long long)(t0 + i) * p.ldy, y[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kLruBatch; ++i) {
+      if (t0 + i < p.S) {
+        lc.step(in[i], S, la);
+        lru_put<T, V>(out + (long long)(t0 + i) * p.C, S, y[i]);
+      }
     }
   }
-  const int t0 = k * p.chunk, t1 = min(p.S, t0 + p.chunk);
-  const T* y = static_cast<const T*>(p.y) + (long long)b * p.S * p.ldy + ch;
-  T* out = static_cast<T*>(p.out) + (long long)b * p.S * p.C + ch;
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-    lc.step(t, S);
-    out[(long long)t * p.C] = from_f32<T>(S * gelu_tanh_f(to_f32(y[(long long)t * p.ldy])));
+  LruChannel<T, V>::store_f32(state, S);
+}
+
+// Pass 1.
+template <typename T, int V>
+__global__ void __launch_bounds__(128) lru_chunk_kernel(const LruParams p) {
+  const int ch = (blockIdx.x * 128 + threadIdx.x) * V, k = blockIdx.y, b = blockIdx.z;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (ch >= p.C) return;
+  const LruChannel<T, V> lc(p, b, ch);
+  float* agg = p.agg + (long long)b * (p.chunks + 1) * 2 * p.C + ch;
+  float S[V], total[V], la[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) S[e] = total[e] = 0.0f;
+  if (k == 0) {                 // pass 2's threads of one channel start from a copy: one of them replaces the state
+    float s0[V];
+    LruChannel<T, V>::load(p.state + (long long)b * p.C + ch, s0);
+    LruChannel<T, V>::store_f32(agg + (long long)p.chunks * 2 * p.C, s0);
   }
-  if (k == p.chunks - 1) p.state[(long long)b * p.C + ch] = S;
+  const int t0 = k * p.chunk, t1 = min(p.S, t0 + p.chunk);
+  typename LruChannel<T, V>::In in[kLruBatch];
+  for (int t = t0; t < t1; t += kLruBatch) {
+#pragma unroll
+    for (int i = 0; i < kLruBatch; ++i)
+      if (t + i < t1) lc.fetch(t + i, in[i]);
+#pragma unroll
+    for (int i = 0; i < kLruBatch; ++i) {
+      if (t + i < t1) {
+        lc.step(in[i], S, la);
+#pragma unroll
+        for (int e = 0; e < V; ++e) total[e] += la[e];
+        float* zt = lc.z + (long long)(t + i) * 2 * p.C;
+        LruChannel<T, V>::store_f32(zt, total);
+        LruChannel<T, V>::store_f32(zt + lc.bw, S);
+      }
+    }
+  }
+  LruChannel<T, V>::store_f32(agg + (long long)k * 2 * p.C, total);
+  LruChannel<T, V>::store_f32(agg + ((long long)k * 2 + 1) * p.C, S);
+}
+
+// Pass 2.
+template <typename T, int V>
+__global__ void __launch_bounds__(128) lru_apply_kernel(const LruParams p) {
+  constexpr bool FAST = sizeof(T) == 2;
+  using Ch = LruChannel<T, V>;
+  const int ch = (blockIdx.x * 128 + threadIdx.x) * V, k = blockIdx.y, b = blockIdx.z;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (ch >= p.C) return;
+  const int bw = p.C / p.blocks;
+  const float* agg = p.agg + (long long)b * (p.chunks + 1) * 2 * p.C + ch;
+  float S0[V];
+  Ch::load(agg + (long long)p.chunks * 2 * p.C, S0);
+#pragma unroll 8
+  for (int j = 0; j < k; ++j) {
+    float total[V], end[V];
+    Ch::load(agg + (long long)j * 2 * p.C, total);
+    Ch::load(agg + ((long long)j * 2 + 1) * p.C, end);
+#pragma unroll
+    for (int e = 0; e < V; ++e) S0[e] += fmaf(expm1_neg_f<FAST>(total[e]), S0[e], end[e]);
+  }
+  const long long row0 = (long long)b * p.S;
+  const float* z = p.z + row0 * 2 * p.C + (long long)(ch / bw) * 2 * bw + ch % bw;
+  const T* yp = static_cast<const T*>(p.y) + row0 * p.ldy + ch;
+  T* out = static_cast<T*>(p.out) + row0 * p.C + ch;
+  const int t0 = k * p.chunk, t1 = min(p.S, t0 + p.chunk);
+  float S[V];
+  for (int t = t0; t < t1; t += kLruBatch) {
+    float total[kLruBatch][V], local[kLruBatch][V], y[kLruBatch][V];
+#pragma unroll
+    for (int i = 0; i < kLruBatch; ++i) {
+      if (t + i < t1) {
+        Ch::load(z + (long long)(t + i) * 2 * p.C, total[i]);
+        Ch::load(z + (long long)(t + i) * 2 * p.C + bw, local[i]);
+        Ch::load(yp + (long long)(t + i) * p.ldy, y[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kLruBatch; ++i) {
+      if (t + i < t1) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) S[e] = fmaf(exp_f<FAST>(total[i][e]), S0[e], local[i][e]);
+        lru_put<T, V>(out + (long long)(t + i) * p.C, S, y[i]);
+      }
+    }
+  }
+  if (k == p.chunks - 1) Ch::store_f32(p.state + (long long)b * p.C + ch, S);
+}
+
+template <typename T, int V>
+static int launch_lru(const LruParams& p, cudaStream_t st) {
+  const unsigned gx = (p.C / V + 127) / 128;
+  if (p.chunks == 1) return counted(1, (int)launch_k(lru_scan_kernel<T, V>, dim3(gx, 1, p.B), dim3(128), (size_t)0, st, p));
+  const dim3 grid(gx, p.chunks, p.B);
+  const int rc = counted(1, (int)launch_k(lru_chunk_kernel<T, V>, grid, dim3(128), (size_t)0, st, p));
+  if (rc) return rc;
+  return counted(1, (int)launch_k(lru_apply_kernel<T, V>, grid, dim3(128), (size_t)0, st, p));
 }
 
 }  // namespace dptb
@@ -212,7 +421,7 @@ using namespace dptb;
 
 struct DptbRecurrentArgs {
   const void* x; const void* taps; const void* conv_bias; float* conv_state; void* u;     // convolution
-  const float* z; const void* br; const void* bi; const void* lam; const void* y;         // recurrence
+  float* z; const void* br; const void* bi; const void* lam; const void* y;         // recurrence
   float* state; void* out; float* agg;
   long long ldx, ldy, agg_floats;
   int B, S, C, K, blocks, chunk, f32;
@@ -226,6 +435,14 @@ extern "C" int dptb_conv_state(const DptbRecurrentArgs* a, void* stream_v) {
   ConvStateParams p;
   p.x = a->x; p.ldx = a->ldx; p.taps = a->taps; p.bias = a->conv_bias; p.state = a->conv_state; p.u = a->u;
   p.B = a->B; p.S = a->S; p.C = a->C; p.K = a->K; p.blocks = a->blocks;
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (!a->f32 && a->K <= 4 && (a->C / a->blocks) % 8 == 0 && a->ldx % 8 == 0 && al16(a->x) && al16(a->conv_bias) && al16(a->u) &&
+      (a->K == 1 || al16(a->conv_state))) {
+    const long long runs = (a->S + kConvRun - 1) / kConvRun * (long long)a->B;
+    const unsigned cy = (a->C / 8 + 127) / 128;
+    if (runs > 0x7fffffff || cy > 65535) return kErrTooLarge;
+    return counted(1, (int)launch_k(conv_state_vec_kernel, dim3((unsigned)runs, cy), dim3(128), (size_t)0, st, p));
+  }
   const int head = a->K - 1 < a->S ? a->K - 1 : a->S;
   const long long units = ((head > 0 ? 1 : 0) + a->S - head) * (long long)a->B;
   const unsigned cy = (a->C + 127) / 128;
@@ -245,15 +462,13 @@ extern "C" int dptb_lru_scan(const DptbRecurrentArgs* a, void* stream_v) {
   p.B = a->B; p.S = a->S; p.C = a->C; p.blocks = a->blocks; p.chunk = a->chunk;
   p.chunks = (a->S + a->chunk - 1) / a->chunk; p.c = a->c;
   if (p.chunks > 65535 || a->B > 65535) return kErrTooLarge;
-  const unsigned gx = (a->C + 127) / 128;
-  if (p.chunks > 1) {
-    if (!a->agg || a->agg_floats < (long long)a->B * (p.chunks + 1) * 2 * a->C) return kErrTooLarge;
-    const dim3 g1(gx, p.chunks - 1, a->B);
-    const int rc = counted(1, (int)(a->f32 ? launch_k(lru_chunk_kernel<float>, g1, dim3(128), (size_t)0, st, p)
-                                           : launch_k(lru_chunk_kernel<__nv_bfloat16>, g1, dim3(128), (size_t)0, st, p)));
-    if (rc) return rc;
-  }
-  const dim3 g2(gx, p.chunks, a->B);
-  return counted(1, (int)(a->f32 ? launch_k(lru_scan_kernel<float>, g2, dim3(128), (size_t)0, st, p)
-                                 : launch_k(lru_scan_kernel<__nv_bfloat16>, g2, dim3(128), (size_t)0, st, p)));
+  if (p.chunks > 1 && (!a->agg || a->agg_floats < (long long)a->B * (p.chunks + 1) * 2 * a->C)) return kErrTooLarge;
+  auto al4 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 3) == 0; };
+  auto al8 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 7) == 0; };
+  const bool pairs = (a->C / a->blocks) % 2 == 0 && a->ldy % 2 == 0 && al4(a->u) && al4(a->y) && al4(a->out) && al8(a->z) &&
+                     al8(a->state) && al8(a->agg);
+  if (a->f32) return launch_lru<float, 1>(p, st);
+  // narrow inputs need the threads more than the wider accesses
+  if (pairs && (long long)a->B * p.chunks * a->C >= 256 * 1024) return launch_lru<__nv_bfloat16, 2>(p, st);
+  return launch_lru<__nv_bfloat16, 1>(p, st);
 }

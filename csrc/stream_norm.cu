@@ -38,13 +38,13 @@ struct StreamParams {
   float eps;
 };
 
-constexpr int kStreamThreads = 128;
+constexpr int kStreamThreads = 256;   // at most
 
 // V consecutive columns per load, NV loads per thread.
 template <typename T, int V, int NV>
 struct StreamRow {
   float v[NV][V];
-  static __device__ __forceinline__ int col(int i) { return (i * kStreamThreads + threadIdx.x) * V; }
+  static __device__ __forceinline__ int col(int i) { return (i * blockDim.x + threadIdx.x) * V; }
   template <typename U>
   static __device__ __forceinline__ void load(const U* p, float (&o)[V]) {
     if constexpr (V == 8) Vec8<U>::load(p, o);
@@ -74,11 +74,19 @@ struct StreamRow {
 #pragma unroll
         for (int k = 0; k < V; ++k) d[k] += t[k];
       }
-      for (int j = 0; j < p.top; ++j) {
-        load(static_cast<const T*>(p.y) + (long long)p.slot[r * p.top + j] * p.D + c, t);
-        const float w = p.w[r * p.top + j];
+      for (int j0 = 0; j0 < p.top; j0 += 4) {      // four experts' rows in flight
+        float yt[4][V], w[4];
 #pragma unroll
-        for (int k = 0; k < V; ++k) d[k] = fmaf(w, t[k], d[k]);
+        for (int j = 0; j < 4; ++j) {
+          const bool on = j0 + j < p.top;
+          const long long at = r * p.top + (on ? j0 + j : 0);
+          w[j] = on ? p.w[at] : 0.0f;
+          load(static_cast<const T*>(p.y) + (long long)p.slot[at] * p.D + c, yt[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int k = 0; k < V; ++k) d[k] = j0 + j < p.top ? fmaf(w[j], yt[j][k], d[k]) : d[k];
       }
 #pragma unroll
       for (int k = 0; k < V; ++k) v[i][k] += d[k];
@@ -177,7 +185,8 @@ __global__ void __launch_bounds__(kStreamThreads) stream_norm_kernel(const Strea
 template <typename T, int V, int NV>
 static int launch_stream(const StreamParams& p, cudaStream_t st) {
   const dim3 grid((unsigned)((p.rows + p.run - 1) / p.run));
-  return counted(1, (int)launch_k(stream_norm_kernel<T, V, NV>, grid, dim3(kStreamThreads), (size_t)0, st, p));
+  const int threads = (((p.D + V * NV - 1) / (V * NV)) + 31) / 32 * 32;
+  return counted(1, (int)launch_k(stream_norm_kernel<T, V, NV>, grid, dim3(threads), (size_t)0, st, p));
 }
 template <typename T>
 static int dispatch_stream(const StreamParams& p, bool vec, cudaStream_t st) {
@@ -186,13 +195,12 @@ static int dispatch_stream(const StreamParams& p, bool vec, cudaStream_t st) {
     if (nv <= 1) return launch_stream<T, 8, 1>(p, st);
     if (nv <= 2) return launch_stream<T, 8, 2>(p, st);
     if (nv <= 4) return launch_stream<T, 8, 4>(p, st);
-    if (nv <= 8) return launch_stream<T, 8, 8>(p, st);
     return kErrUnsupported;
   }
   const int nv = (p.D + kStreamThreads - 1) / kStreamThreads;
-  if (nv <= 4) return launch_stream<T, 1, 4>(p, st);
-  if (nv <= 16) return launch_stream<T, 1, 16>(p, st);
-  if (nv <= 64) return launch_stream<T, 1, 64>(p, st);
+  if (nv <= 2) return launch_stream<T, 1, 2>(p, st);
+  if (nv <= 8) return launch_stream<T, 1, 8>(p, st);
+  if (nv <= 32) return launch_stream<T, 1, 32>(p, st);
   return kErrUnsupported;
 }
 

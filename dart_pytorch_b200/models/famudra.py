@@ -11,6 +11,7 @@ captured in a CUDA graph, once per cache, and replayed.
 """
 from __future__ import annotations
 
+import gc
 import os
 from dataclasses import dataclass
 from typing import List, Optional, Sequence, Tuple
@@ -219,8 +220,16 @@ class Famudra(CausalLMMixin, Module):
             torch.cuda.synchronize()
             launches = lib.dptb_launch_count()
             graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph, stream=s):
-                logits = body()
+            # an unreachable older graph must not be destroyed while this one is being recorded
+            gc.collect()
+            collecting = gc.isenabled()
+            gc.disable()
+            try:
+                with torch.cuda.graph(graph, stream=s):
+                    logits = body()
+            finally:
+                if collecting:
+                    gc.enable()
         torch.cuda.current_stream().wait_stream(s)
         cache.graph = (graph, tokens, logits, int(lib.dptb_launch_count() - launches))
 

@@ -94,7 +94,7 @@ class HybridCache:
         # per layer run: rows per expert and places handed out, zeroed at the start of a step
         self.counters = torch.zeros(max(1, len(states)), max(1, counters), dtype=torch.int32, device=device)
         self.capacity = 0
-        self.plan: Dict[object, object] = {}
+        self.plan: Dict[int, torch.Tensor] = {}           # attention workspace by rows of a step
         self.graph = None
         self.ensure(max(1, max_len))
 
@@ -110,18 +110,15 @@ class HybridCache:
         self.graph = None
 
     def attn_workspace(self, rows: int, H: int, R: int, max_keys: int):
-        """(slices, workspace, counters) of the latent attention kernel, one allocation per shape."""
+        """(slices, workspace) of the latent attention kernel; all layers share one workspace."""
         from ..ops import hybrid as Y
-        splits, floats, ctrs = Y.latent_attn_plan(rows, H, R, max_keys, self.dtype == torch.float32)
+        splits, floats = Y.latent_attn_plan(rows, H, R, max_keys, self.dtype == torch.float32)
         if splits <= 1:
-            return 1, None, None
-        key = (rows, H, R)
-        got = self.plan.get(key)
-        if got is None or got[0].numel() < floats:
-            got = (torch.empty(floats, dtype=torch.float32, device=self.device),
-                   torch.zeros(ctrs, dtype=torch.int32, device=self.device))
-            self.plan[key] = got
-        return splits, got[0], got[1]
+            return 1, None
+        got = self.plan.get(rows)
+        if got is None or got.numel() < floats:
+            got = self.plan[rows] = torch.empty(floats, dtype=torch.float32, device=self.device)
+        return splits, got
 
     def advance(self, n: int) -> None:
         self.seq_len += n
@@ -288,9 +285,8 @@ class LatentAttention(_Packed):
         q = F.linear(cq, self.w_uq)
         ql = torch.empty(M, H * R, dtype=q.dtype, device=q.device)
         Y.grouped_gemm(Y.grouped_segment(q, pack["uk_t"], ql, groups=H, N_=R, K=dk, x_col_stride=dk, out_col_stride=R))
-        splits, ws, ctrs = ctx.cache.attn_workspace(M, H, R, ctx.max_keys)
-        ol = Y.latent_attn(ql, state.buf, ctx.B, ctx.S, H, ctx.pos, self.scale, pos_ptr=ctx.pos_ptr, splits=splits, ws=ws,
-                           counters=ctrs)
+        splits, ws = ctx.cache.attn_workspace(M, H, R, ctx.max_keys)
+        ol = Y.latent_attn(ql, state.buf, ctx.B, ctx.S, H, ctx.pos, self.scale, pos_ptr=ctx.pos_ptr, splits=splits, ws=ws)
         o = torch.empty(M, H * dv, dtype=q.dtype, device=q.device)
         Y.grouped_gemm(Y.grouped_segment(ol, self.w_uv.detach(), o, groups=H, N_=dv, K=R, x_col_stride=R,
                                          out_col_stride=dv))

@@ -22,9 +22,8 @@ class GroupedSegArgs(ctypes.Structure):
 
 
 class LatentArgs(ctypes.Structure):
-    _fields_ = [("d", P), ("gq", P), ("gc", P), ("cq", P), ("c_new", P), ("q", P), ("o", P), ("ws", P), ("counters", P),
-                ("cache", P), ("pos_ptr", P), ("ldd", L), ("ws_floats", L), ("B", I), ("S", I), ("H", I), ("Rq", I),
-                ("R", I), ("cap", I), ("pos", I), ("splits", I), ("num_counters", I), ("f32", I), ("force_simt", I),
+    _fields_ = [("d", P), ("gq", P), ("gc", P), ("cq", P), ("c_new", P), ("q", P), ("o", P), ("ws", P), ("cache", P), ("pos_ptr", P), ("ldd", L), ("ws_floats", L), ("B", I), ("S", I), ("H", I), ("Rq", I),
+                ("R", I), ("cap", I), ("pos", I), ("splits", I), ("f32", I), ("force_simt", I),
                 ("eps", F), ("scale", F)]
 
 
@@ -143,22 +142,21 @@ def latent_norm_append(d: torch.Tensor, gq, gc, cache, B: int, S: int, pos: int,
 
 
 def latent_attn_plan(rows: int, H: int, R: int, max_keys: int, f32: bool):
-    """(key slices, workspace floats, counters) for ``rows`` queries over up to ``max_keys`` cached tokens."""
+    """(key slices, workspace floats) for ``rows`` queries over up to ``max_keys`` cached tokens."""
     lib = _lib()
     s = lib.dptb_latent_attn_splits(rows, H, R, max_keys, int(f32))
-    return s, int(lib.dptb_latent_attn_ws_floats(rows, H, R, s)), rows * ((H + 15) // 16)
+    return s, int(lib.dptb_latent_attn_ws_floats(rows, H, R, s))
 
 
 def latent_attn(q: torch.Tensor, cache: torch.Tensor, B: int, S: int, H: int, pos: int, scale: float,
                 pos_ptr: Optional[torch.Tensor] = None, splits: int = 1, ws: Optional[torch.Tensor] = None,
-                counters: Optional[torch.Tensor] = None, force_simt: bool = False) -> torch.Tensor:
+                force_simt: bool = False) -> torch.Tensor:
     """Causal attention in latent space: ``q [B*S, H*R]`` against ``cache [B, cap, R]``, query ``s`` seeing the rows up to
     ``pos + s``; returns ``[B*S, H*R]``."""
     a = _latent_args(cache, B, S, pos, pos_ptr)
     out = torch.empty_like(q)
     a.q, a.o, a.H, a.scale = _same(q, cache.dtype, [B * S, H * a.R], "q"), out.data_ptr(), H, scale
-    a.splits, a.ws, a.counters = splits, N.ptr(ws), N.ptr(counters)
-    a.ws_floats, a.num_counters = (0 if ws is None else ws.numel()), (0 if counters is None else counters.numel())
+    a.splits, a.ws, a.ws_floats = splits, N.ptr(ws), 0 if ws is None else ws.numel()
     a.force_simt = int(force_simt)
     N.check(_lib().dptb_latent_attn(ctypes.byref(a), N.stream_ptr()), "latent_attn")
     return out
@@ -187,7 +185,7 @@ def conv_state(x: torch.Tensor, taps, bias, state: torch.Tensor, B: int, S: int,
 
 def lru_scan(u, z, br, bi, lam, y, state, B: int, S: int, blocks: int, c: float, chunk: int = LRU_CHUNK) -> torch.Tensor:
     """Gated linear recurrence from ``state [B, C]`` (fp32, updated) and its product with ``gelu_tanh(y)``; ``z`` holds the
-    fp32 gate products ``[B*S, blocks, 2, C/blocks]``.  Returns ``[B*S, C]``."""
+    fp32 gate products ``[B*S, blocks, 2, C/blocks]`` and is used as scratch.  Returns ``[B*S, C]``."""
     a = RecurrentArgs()
     C = lam.numel()
     out = torch.empty(B * S, C, dtype=y.dtype, device=y.device)
@@ -224,7 +222,10 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, counters: torch.T
     a.x, a.ldx, a.router = _same(x, router.dtype, [T, D], "x"), D, _same(router, x.dtype, [E, D], "router")
     if (T > ROUTER_KERNEL_ROWS and not a.f32) or 4 * (D + E) > 48 * 1024:
         logits = torch.empty(T, E, dtype=torch.float32, device=x.device)
-        K.gemm(x, router, logits, trans_b=True)
+        if a.f32:
+            K.gemm(x, router, logits, trans_b=True)
+        else:       # few output features: narrow token tiles put the product on all SMs
+            grouped_gemm(grouped_segment(x, router, logits, groups=1, N_=E, K=D, rows_hint=64))
         a.logits, a.ld_logits = logits.data_ptr(), E
     a.idx, a.w, a.count = idx.data_ptr(), w.data_ptr(), counters.data_ptr()
     a.T, a.D, a.E, a.top = T, D, E, top
