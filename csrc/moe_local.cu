@@ -19,41 +19,48 @@ namespace dptb {
 constexpr int kMoeMaxExperts = 1024;
 constexpr int kMoeMaxTop = 32;
 
-// One warp chooses from `sel` (shared memory, E values, consumed).  Ties resolve to the lowest index.
+// Floats as unsigned integers of the same order, and back.
+__device__ __forceinline__ uint32_t ordered_bits(float v) {
+  const uint32_t u = __float_as_uint(v);
+  return (u & 0x80000000u) ? ~u : u | 0x80000000u;
+}
+__device__ __forceinline__ float from_ordered(uint32_t k) {
+  return __uint_as_float((k & 0x80000000u) ? k & 0x7fffffffu : ~k);
+}
+
+// One warp chooses the `top` largest of `sel` (shared memory, E values, consumed).  Ties resolve to the lowest index.  A
+// lane keeps the best of its own experts (lane, lane + 32, ...); a round is two warp reductions, and only the winner's
+// lane looks through its experts again.
 __device__ __forceinline__ void choose_top(float* sel, int E, int top, int lane, int* idx, float* w, int* count) {
+  constexpr uint32_t kNone = 0xffffffffu;
+  auto best = [&](uint32_t& key, uint32_t& at) {
+    key = 0;
+    at = kNone;
+    for (int e = lane; e < E; e += 32) {
+      const uint32_t k = ordered_bits(sel[e]);
+      if (at == kNone || k > key) {
+        key = k;
+        at = e;
+      }
+    }
+  };
+  uint32_t key, at;
+  best(key, at);
   float mine = 0.0f, first = 0.0f, sum = 0.0f;
   for (int j = 0; j < top; ++j) {
-    float bv = -INFINITY;
-    int bi = -1;
-    for (int e = lane; e < E; e += 32) {
-      const float v = sel[e];
-      if (bi < 0 || v > bv) {
-        bv = v;
-        bi = e;
-      }
-    }
-    if (bi < 0) bi = E;       // lanes without an expert never win
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (bi >= E || (oi < E && (ov > bv || (ov == bv && oi < bi)))) {
-        bv = ov;
-        bi = oi;
-      }
-    }
-    bi = __shfl_sync(0xffffffffu, bi, 0);     // one answer even when NaNs broke the ordering
-    bv = __shfl_sync(0xffffffffu, bv, 0);
-    if (j == 0) first = bv;
-    const float ex = expf(bv - first);
+    const uint32_t k = __reduce_max_sync(0xffffffffu, key);
+    const uint32_t e = __reduce_min_sync(0xffffffffu, key == k ? at : kNone);
+    const float v = from_ordered(k);
+    if (j == 0) first = v;
+    const float ex = expf(v - first);
     sum += ex;
     if (lane == j) mine = ex;
-    if (lane == 0) {
-      idx[j] = bi;
-      sel[bi] = -INFINITY;
-      atomicAdd(&count[bi], 1);
+    if (at == e) {
+      idx[j] = (int)e;
+      sel[e] = -INFINITY;
+      atomicAdd(&count[e], 1);
+      best(key, at);
     }
-    __syncwarp();
   }
   if (lane < top) w[lane] = mine / sum;
 }
