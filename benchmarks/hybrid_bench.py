@@ -92,7 +92,7 @@ def measure_llama(s, steps: int, warmup: int) -> dict:
     from dart_pytorch_b200.models.llama import LlamaConfig
     from dart_pytorch_b200.parallel.tp_llama import TPLlamaEngine
     if not dist.is_initialized():
-        os.environ["NCCL_DEBUG"] = "WARN"          # standard output carries one JSON line
+        os.environ["NCCL_DEBUG"] = "NONE"          # standard output carries one JSON line
         os.environ.setdefault("MASTER_ADDR", "127.0.0.1")
         os.environ.setdefault("MASTER_PORT", "29577")
         dist.init_process_group("nccl", rank=0, world_size=1, device_id=torch.device("cuda", torch.cuda.current_device()))

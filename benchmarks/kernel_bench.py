@@ -182,6 +182,7 @@ def build_hybrid_cases(dev):
     from dart_pytorch_b200.nn.hybrid import DroplessMoE
     from dart_pytorch_b200.ops import decode as Dk
     from dart_pytorch_b200.ops import hybrid as Y
+    from dart_pytorch_b200.parallel import ep as EP
     bf = dict(device=dev, dtype=torch.bfloat16)
     f32 = dict(device=dev, dtype=torch.float32)
     D, H, hd, Rq, R, C, G, E, top, ff, sff, V = 2048, 16, 128, 768, 512, 2560, 10, 64, 6, 1024, 2048, 32768
@@ -230,6 +231,12 @@ def build_hybrid_cases(dev):
         flops = 2.0 * rows * D * (top * ff + sff)
         add(tag + "experts_up", run_up, wb + 2 * rows * (top * (D + ff) + D + sff), flops)
         add(tag + "experts_down", run_down, wb + 2 * rows * (top * (D + ff) + D + sff), flops)
+        like_logits = torch.empty(rows, E, **bf)
+
+        def like_route(x=x, like_logits=like_logits, rows=rows):    # the expert-parallel MoE layer's router
+            K.gemm(x, router, like_logits, trans_b=True)
+            EP.slots(EP.route(like_logits, top)[1], E, rows)
+        add("like_" + tag + "route", like_route, 2 * rows * D)
         add(tag + "route", lambda x=x, ctr=ctr: Y.moe_route(x, router, top, ctr), 2 * rows * D)
 
         def place(x=x, idx=idx, ctr=ctr, base=base):

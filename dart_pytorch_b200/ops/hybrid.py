@@ -163,7 +163,10 @@ def latent_attn(q: torch.Tensor, cache: torch.Tensor, B: int, S: int, H: int, po
 
 
 # --------------------------------------------------------------------------- convolution + recurrence
-LRU_CHUNK = 64
+def lru_chunk(S: int) -> int:
+    """Tokens per chunk of the two-pass recurrence: about 0.7 sqrt(S), where the steps inside a chunk and the chunks to fold
+    balance (measured between 512 and 8192 tokens)."""
+    return 16 if S <= 1024 else 32 if S <= 4096 else 64 if S <= 32768 else 128
 
 
 def conv_state(x: torch.Tensor, taps, bias, state: torch.Tensor, B: int, S: int, blocks: int) -> torch.Tensor:
@@ -183,12 +186,14 @@ def conv_state(x: torch.Tensor, taps, bias, state: torch.Tensor, B: int, S: int,
     return u
 
 
-def lru_scan(u, z, br, bi, lam, y, state, B: int, S: int, blocks: int, c: float, chunk: int = LRU_CHUNK) -> torch.Tensor:
+def lru_scan(u, z, br, bi, lam, y, state, B: int, S: int, blocks: int, c: float,
+             chunk: Optional[int] = None) -> torch.Tensor:
     """Gated linear recurrence from ``state [B, C]`` (fp32, updated) and its product with ``gelu_tanh(y)``; ``z`` holds the
     fp32 gate products ``[B*S, blocks, 2, C/blocks]`` and is used as scratch.  Returns ``[B*S, C]``."""
     a = RecurrentArgs()
     C = lam.numel()
     out = torch.empty(B * S, C, dtype=y.dtype, device=y.device)
+    chunk = lru_chunk(S) if chunk is None else chunk
     chunks = (S + chunk - 1) // chunk
     agg = torch.empty(B * (chunks + 1) * 2 * C, dtype=torch.float32, device=y.device) if chunks > 1 else None
     f32 = _f32(y)
