@@ -17,7 +17,14 @@
 // the splits itself (arrival counter), so one kernel runs per call (attn_decode_merge_kernel remains for shapes beyond
 // the counter table).
 // The kernel is memory-bound by design: the roofline is the KV bytes over HBM bandwidth.
+//
+// The windowed form (WIN) reads a ring of token rows (position p is row p % ring), of which a query sees the last `window`
+// positions, and before them pooled rows (one per block of `pool` tokens that has left the window).  Heads may be smaller than
+// HD (multiples of 8), keys and values of different sizes; a sink (a score without a key) joins the final sum, and outputs can
+// be turned by the query's position.
 #include <cuda_bf16.h>
+
+#include <initializer_list>
 
 #include "common/host.h"
 #include "common/ptx.cuh"
@@ -43,6 +50,12 @@ struct DecodeArgs {
                              // captured CUDA graph can be replayed as the sequence grows)
   int cap;                   // cache rows per sequence: no key at or beyond it is ever read
   int fused_merge;           // the last split CTA of a (query row, kv head) merges the partials itself
+  // windowed form
+  const __nv_bfloat16* k_pool;   // [B, pool_rows, Hkv * dk]
+  const __nv_bfloat16* v_pool;   // [B, pool_rows, Hkv * dv]
+  const __nv_bfloat16* sink;     // [Hq] or null
+  const float2* rot;             // [positions, dv / 2] or null
+  int window, pool, pool_rows, ring, dk, dv;
 };
 
 __device__ __forceinline__ void unpack_bf16x8(const uint4& u, float (&f)[8]) {
@@ -73,6 +86,10 @@ __device__ __forceinline__ void cp_async_16(void* smem_dst, const void* gsrc) {
   const uint32_t d = static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst));
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(gsrc) : "memory");
 }
+__device__ __forceinline__ void cp_async_16_or_zero(void* smem_dst, const void* gsrc, bool valid) {
+  const uint32_t d = static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst));
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(gsrc), "r"(valid ? 16 : 0) : "memory");
+}
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
@@ -84,7 +101,18 @@ constexpr int kDecCounters = 1 << 16;
 __device__ unsigned int g_dec_counters[kDecCounters];
 constexpr int kDecMaxFusedSplits = 64;
 
-template <int HD, int GP>
+// The last step of an output feature in the windowed form: turned back by the query's position.  Whole warps call it.
+__device__ __forceinline__ void decode_store_windowed(const DecodeArgs& a, int bs, int head, int d, int pos, float v) {
+  const float u = __shfl_xor_sync(0xffffffffu, v, 1);
+  if (d >= a.dv) return;
+  if (a.rot) {
+    const float2 cs = a.rot[(long long)pos * (a.dv / 2) + d / 2];
+    v = d & 1 ? v * cs.x - u * cs.y : v * cs.x + u * cs.y;
+  }
+  a.o[(long long)bs * a.ldo + (long long)head * a.dv + d] = __float2bfloat16(v);
+}
+
+template <int HD, int GP, bool WIN>
 __global__ void __launch_bounds__(kDecWarps * 32, GP <= 4 ? 3 : 2)
 attn_decode_kernel(const DecodeArgs a) {
   constexpr int LPK = HD / 8;                // lanes per key
@@ -102,7 +130,14 @@ attn_decode_kernel(const DecodeArgs a) {
   const int sl = lane & (LPK - 1), sg0 = lane & ~(LPK - 1);   // lane within the sub-group, first lane of the sub-group
   const int q_off = a.pos_ptr ? *a.pos_ptr : a.q_offset;
   const int sk = a.pos_ptr ? q_off + a.Sq : a.Sk;
-  const int visible = min(min(sk, a.cap), q_off + sq + 1);     // causal limit for this query row
+  const int q_pos = q_off + sq;
+  const int lo = WIN ? max(0, q_pos - a.window + 1) : 0;       // first token of the window
+  const int left = q_pos - a.window + 1;
+  const int blocks = WIN && a.pool > 0 && left >= a.pool ? min(left / a.pool, a.pool_rows) : 0;
+  const int slot0 = WIN ? lo % a.ring : 0;
+  // keys of this query row: pooled rows, then the window; or everything up to its own position
+  const int visible = WIN ? blocks + q_pos - lo + 1 : min(min(sk, a.cap), q_pos + 1);
+  const int dk = WIN ? a.dk : HD, dv = WIN ? a.dv : HD;
   const int per = (visible + a.splits - 1) / a.splits;
   const int j0 = split * per, j1 = min(visible, j0 + per);
 
@@ -110,12 +145,12 @@ attn_decode_kernel(const DecodeArgs a) {
   __shared__ float s_acc[kDecWarps][GP][HD];
 
   f32x2 qv[GP][4];
-  const __nv_bfloat16* qrow = a.q + (long long)bs * a.ldq + (long long)g * G * HD + sl * 8;
+  const __nv_bfloat16* qrow = a.q + (long long)bs * a.ldq + (long long)g * G * dk + sl * 8;
   const f32x2 scale2 = f2_splat(a.scale);
 #pragma unroll
   for (int h = 0; h < GP; ++h) {
-    if (h < G) {
-      unpack_bf16x8_f2(*reinterpret_cast<const uint4*>(qrow + h * HD), qv[h]);
+    if (h < G && (!WIN || sl * 8 < dk)) {
+      unpack_bf16x8_f2(*reinterpret_cast<const uint4*>(qrow + h * dk), qv[h]);
 #pragma unroll
       for (int e = 0; e < 4; ++e) qv[h][e] = f2_mul(qv[h][e], scale2);
     } else {
@@ -134,6 +169,13 @@ attn_decode_kernel(const DecodeArgs a) {
   }
   const __nv_bfloat16* kb = a.k + (long long)b * a.kv_batch_stride + (long long)g * HD;
   const __nv_bfloat16* vb = a.v + (long long)b * a.kv_batch_stride + (long long)g * HD;
+  const int ldk = a.Hkv * dk, ldv = a.Hkv * dv;                // windowed form: rows of the ring and of the pooled blocks
+  if constexpr (WIN) {
+    kb = a.k + (long long)b * a.ring * ldk + g * dk;
+    vb = a.v + (long long)b * a.ring * ldv + g * dv;
+  }
+  const __nv_bfloat16* kpb = WIN ? a.k_pool + (long long)b * a.pool_rows * ldk + g * dk : nullptr;
+  const __nv_bfloat16* vpb = WIN ? a.v_pool + (long long)b * a.pool_rows * ldv + g * dv : nullptr;
   uint4* ring = dec_ring + warp * kWarpChunks;   // [stage][K | V][16 rows][LPK chunks]
   const int sg = lane / LPK;
   const int rounds = (j1 - j0 + kDecRound - 1) / kDecRound;   // of this CTA; warp w takes rounds w, w + 4, ...
@@ -145,9 +187,20 @@ attn_decode_kernel(const DecodeArgs a) {
     for (int it = 0; it < kStageChunks / 32; ++it) {
       const int c = it * 32 + lane;
       const int key = min(key0 + c / LPK, j1 - 1);
-      const long long off = (long long)key * a.ldkv + (c % LPK) * 8;
-      cp_async_16(dst + c, kb + off);
-      cp_async_16(dst + kStageChunks + c, vb + off);
+      if constexpr (WIN) {
+        const bool pooled = key < blocks;
+        int r = pooled ? key : slot0 + key - blocks;
+        if (!pooled && r >= a.ring) r -= a.ring;
+        const int f = (c % LPK) * 8;
+        const __nv_bfloat16* kr = (pooled ? kpb : kb) + (long long)r * ldk;
+        const __nv_bfloat16* vr = (pooled ? vpb : vb) + (long long)r * ldv;
+        cp_async_16_or_zero(dst + c, f < dk ? kr + f : kr, f < dk);
+        cp_async_16_or_zero(dst + kStageChunks + c, f < dv ? vr + f : vr, f < dv);
+      } else {
+        const long long off = (long long)key * a.ldkv + (c % LPK) * 8;
+        cp_async_16(dst + c, kb + off);
+        cp_async_16(dst + kStageChunks + c, vb + off);
+      }
     }
     cp_async_commit();
   };
@@ -246,7 +299,14 @@ attn_decode_kernel(const DecodeArgs a) {
       ll += s_l[w][h] * c;
       oo += s_acc[w][h][d] * c;
     }
-    if (a.splits == 1) {
+    if (WIN && a.splits == 1) {
+      if (a.sink) {
+        const float s = __bfloat162float(a.sink[g * G + h]), m1 = fmaxf(mm, s), c = __expf(mm - m1);
+        ll = ll * c + __expf(s - m1);
+        oo *= c;
+      }
+      decode_store_windowed(a, bs, g * G + h, d, q_pos, oo / ll);
+    } else if (a.splits == 1) {
       a.o[(long long)bs * a.ldo + (long long)(g * G + h) * HD + d] = __float2bfloat16(ll > 0.0f ? oo / ll : 0.0f);
     } else {
       float* w = a.ws + ((((long long)bs * a.Hkv + g) * a.splits + split) * G + h) * (HD + 2);
@@ -328,9 +388,18 @@ attn_decode_kernel(const DecodeArgs a) {
 #pragma unroll
   for (int k = 0; k < NO; ++k) {
     const int idx = threadIdx.x + k * (kDecWarps * 32);
-    if (idx / HD < G)
+    if (idx / HD >= G) continue;
+    if constexpr (WIN) {
+      if (a.sink) {
+        const float s = __bfloat162float(a.sink[g * G + hh[k]]), m1 = fmaxf(mm[k], s), c = __expf(mm[k] - m1);
+        ll[k] = ll[k] * c + __expf(s - m1);
+        oo[k] *= c;
+      }
+      decode_store_windowed(a, bs, g * G + hh[k], idx % HD, q_pos, oo[k] / ll[k]);
+    } else {
       a.o[(long long)bs * a.ldo + (long long)(g * G + idx / HD) * HD + idx % HD] =
           __float2bfloat16(ll[k] > 0.0f ? oo[k] / ll[k] : 0.0f);
+    }
   }
 }
 
@@ -447,6 +516,27 @@ extern "C" int dptb_attn_decode_splits_hd(int B, int Sq, int Hkv, int Sk, int he
   return decode_splits(B, Sq, Hkv, Sk, head_dim);
 }
 
+// ring: two stages of 16 K rows and 16 V rows per warp
+template <int HD, int GP, bool WIN>
+static cudaError_t decode_launch_gp(const DecodeArgs& a, dim3 grid, cudaStream_t st) {
+  constexpr int kRing = kDecWarps * 4 * kDecRound * HD * 2;
+  static bool attr_set = false;
+  if (!attr_set) {
+    const cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<HD, GP, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               kRing);
+    if (e != cudaSuccess) return e;
+    attr_set = true;
+  }
+  return launch_k(attn_decode_kernel<HD, GP, WIN>, grid, dim3(kDecWarps * 32), kRing, st, a);
+}
+template <int HD, bool WIN>
+static cudaError_t decode_launch(const DecodeArgs& a, int gp, dim3 grid, cudaStream_t st) {
+  if (gp == 1) return decode_launch_gp<HD, 1, WIN>(a, grid, st);
+  if (gp == 2) return decode_launch_gp<HD, 2, WIN>(a, grid, st);
+  if (gp == 4) return decode_launch_gp<HD, 4, WIN>(a, grid, st);
+  return decode_launch_gp<HD, 8, WIN>(a, grid, st);
+}
+
 extern "C" int dptb_attn_decode(const DptbDecodeArgs* h, void* stream) {
   auto st = static_cast<cudaStream_t>(stream);
   if (h->B <= 0 || h->Sq <= 0 || h->Sk <= 0) return 0;
@@ -456,7 +546,7 @@ extern "C" int dptb_attn_decode(const DptbDecodeArgs* h, void* stream) {
   if ((h->ldkv % 8) || (h->kv_batch_stride % 8) || (h->ldq % 8) || (reinterpret_cast<uintptr_t>(h->k) & 15) ||
       (reinterpret_cast<uintptr_t>(h->v) & 15) || (reinterpret_cast<uintptr_t>(h->q) & 15))
     return kErrBadShape;
-  DecodeArgs a;
+  DecodeArgs a = {};
   a.q = static_cast<const __nv_bfloat16*>(h->q);
   a.k = static_cast<const __nv_bfloat16*>(h->k);
   a.v = static_cast<const __nv_bfloat16*>(h->v);
@@ -473,24 +563,7 @@ extern "C" int dptb_attn_decode(const DptbDecodeArgs* h, void* stream) {
   const int G = a.Hq / a.Hkv;
   a.fused_merge = (a.splits > 1 && a.splits <= kDecMaxFusedSplits && (long long)a.B * a.Sq * a.Hkv <= kDecCounters) ? 1 : 0;
   const int gp = G <= 1 ? 1 : G <= 2 ? 2 : G <= 4 ? 4 : 8;
-  // ring: two stages of 16 K rows and 16 V rows per warp
-#define DPTB_DEC(HDV, GPV)                                                                                            \
-  do {                                                                                                                \
-    constexpr int kRing = kDecWarps * 4 * kDecRound * HDV * 2;                                                        \
-    static bool attr_set = false;                                                                                     \
-    if (!attr_set) {                                                                                                  \
-      DPTB_CUDA_OK(cudaFuncSetAttribute(attn_decode_kernel<HDV, GPV>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
-                                        kRing));                                                                      \
-      attr_set = true;                                                                                                \
-    }                                                                                                                 \
-    DPTB_CUDA_OK(launch_k(attn_decode_kernel<HDV, GPV>, grid, dim3(kDecWarps * 32), kRing, st, a));                   \
-  } while (0)
-  if (h->head_dim == 128) {
-    if (gp == 1) DPTB_DEC(128, 1); else if (gp == 2) DPTB_DEC(128, 2); else if (gp == 4) DPTB_DEC(128, 4); else DPTB_DEC(128, 8);
-  } else {
-    if (gp == 1) DPTB_DEC(64, 1); else if (gp == 2) DPTB_DEC(64, 2); else if (gp == 4) DPTB_DEC(64, 4); else DPTB_DEC(64, 8);
-  }
-#undef DPTB_DEC
+  DPTB_CUDA_OK((h->head_dim == 128 ? decode_launch<128, false>(a, gp, grid, st) : decode_launch<64, false>(a, gp, grid, st)));
   DPTB_CUDA_OK(cudaGetLastError());
   if (a.splits > 1 && !a.fused_merge) {
     dim3 mg(a.Hq, a.B * a.Sq);
@@ -499,6 +572,56 @@ extern "C" int dptb_attn_decode(const DptbDecodeArgs* h, void* stream) {
     return counted(2, (int)cudaGetLastError());
   }
   return counted(1, (int)cudaGetLastError());
+}
+
+struct DptbWindowDecodeArgs {
+  const void* q;              // [B * S, H * dk]
+  const void* k;              // [B, ring, G * dk]
+  const void* v;              // [B, ring, G * dv]
+  const void* k_pool;         // [B, pool_rows, G * dk] or null
+  const void* v_pool;
+  const void* sink;
+  const void* rot;
+  void* o;                    // [B * S, H * dv]
+  float* ws;
+  const int* pos_ptr;
+  long long ws_floats;
+  int B, S, H, G, dk, dv, ring, window, pool, pool_rows, pos, splits;
+  float scale;
+};
+
+// Windowed attention of a short step straight from the ring.
+extern "C" int dptb_window_attn_decode(const DptbWindowDecodeArgs* h, void* stream) {
+  auto st = static_cast<cudaStream_t>(stream);
+  if (h->B <= 0 || h->S <= 0) return 0;
+  if (h->G <= 0 || h->H % h->G || h->dk <= 0 || h->dv <= 0 || h->window < 1 || h->window + h->S - 1 > h->ring) return kErrBadShape;
+  const int G = h->H / h->G, hd = h->dk > h->dv ? h->dk : h->dv;
+  if (G > kMaxGroup || h->dk % 8 || h->dv % 8 || hd > 128 || (long long)h->B * h->S > 65535) return kErrUnsupported;
+  if (h->pool > 0 && (!h->k_pool || !h->v_pool)) return kErrBadShape;
+  for (const void* q : {h->q, h->k, h->v, h->k_pool, h->v_pool})
+    if (reinterpret_cast<uintptr_t>(q) & 15) return kErrBadShape;
+  DecodeArgs a = {};
+  a.q = static_cast<const __nv_bfloat16*>(h->q);
+  a.k = static_cast<const __nv_bfloat16*>(h->k);
+  a.v = static_cast<const __nv_bfloat16*>(h->v);
+  a.k_pool = static_cast<const __nv_bfloat16*>(h->k_pool);
+  a.v_pool = static_cast<const __nv_bfloat16*>(h->v_pool);
+  a.sink = static_cast<const __nv_bfloat16*>(h->sink);
+  a.rot = static_cast<const float2*>(h->rot);
+  a.o = static_cast<__nv_bfloat16*>(h->o);
+  a.ws = h->ws;
+  a.ldq = (long long)h->H * h->dk; a.ldo = (long long)h->H * h->dv;
+  a.B = h->B; a.Sq = h->S; a.Hq = h->H; a.Hkv = h->G; a.q_offset = h->pos; a.scale = h->scale; a.pos_ptr = h->pos_ptr;
+  a.window = h->window; a.pool = h->pool; a.pool_rows = h->pool_rows; a.ring = h->ring; a.dk = h->dk; a.dv = h->dv;
+  a.splits = h->splits < 1 ? 1 : h->splits;
+  // the splits are merged by the last CTA of a row only
+  if (a.splits > kDecMaxFusedSplits || (a.splits > 1 && (long long)h->B * h->S * h->G > kDecCounters)) return kErrTooLarge;
+  a.fused_merge = a.splits > 1;
+  const int HD = hd <= 64 ? 64 : 128;
+  if (a.splits > 1 && (!a.ws || h->ws_floats < dptb_attn_decode_ws_floats(a.B, a.Sq, a.Hq, HD, a.splits))) return kErrTooLarge;
+  const dim3 grid(a.splits, a.Hkv, a.B * a.Sq);
+  const int gp = G <= 1 ? 1 : G <= 2 ? 2 : G <= 4 ? 4 : 8;
+  return counted(1, (int)(HD == 128 ? decode_launch<128, true>(a, gp, grid, st) : decode_launch<64, true>(a, gp, grid, st)));
 }
 
 extern "C" int dptb_rope_kv_append(void* qkv, long long ld, void* kc, void* vc, long long ldkv,

@@ -22,7 +22,15 @@
 //
 // The precise form (PREC) walks tiles of 64 keys and keeps every softmax weight as a high and a low bf16 part (16 mantissa
 // bits): both parts of a 64-key tile take the room one part of a 128-key tile has, and P V is two products.
+//
+// The windowed form (WIN) sees the last `window` tokens and, in front of them, pooled rows of a second pair of K / V buffers
+// (one row per block of `pool` tokens, visible once the whole block has left the window); tiles of pooled rows are walked
+// first, then the token tiles that the window touches.  A sink (a score without a key) starts the running sum.  Heads may have
+// any size up to HD that is a multiple of 8, keys and values of different sizes: the tensor maps fill the rest with zeros.
+// Outputs can be turned by the query's position (pairs (2m, 2m + 1), a table of cosines and sines) on the way out.
 #include <cuda_bf16.h>
+
+#include <initializer_list>
 
 #include "common/host.h"
 #include "common/ptx.cuh"
@@ -38,6 +46,12 @@ struct AttnFwdParams {
   int q_offset;           // key j is visible to query i when j <= i + q_offset (causal)
   float scale_log2;       // softmax scale * log2(e)
   int num_q_blocks;
+  // windowed form
+  int window, pool, pool_rows;
+  int pos;                // position of query row 0; row i of K / V is position i + pos - q_offset
+  int dv;
+  const __nv_bfloat16* sink;    // [Hq] or null
+  const float2* rot;            // [positions, dv / 2] (cos, sin) or null
 };
 
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -83,10 +97,11 @@ struct AttnFwdSmem {
   static_assert(kTotal <= 227 * 1024, "attention forward: shared memory budget");
 };
 
-template <int HD, int NQ, int KST, int VST, bool PREC>
+template <int HD, int NQ, int KST, int VST, bool PREC, bool WIN>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                const __grid_constant__ CUtensorMap tmV, const AttnFwdParams p) {
+                const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmPK,
+                const __grid_constant__ CUtensorMap tmPV, const AttnFwdParams p) {
   using L = AttnFwdSmem<HD, NQ, KST, VST, PREC>;
   constexpr int kAttnBN = L::kBN;
   constexpr int kChunks = HD / 64;            // 64-column (128-byte) chunks per head row
@@ -116,9 +131,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   const int kv_head = head / (p.Hq / p.Hkv);
   const int q_row0 = qb * (NQ * kAttnBM);
 
-  // Number of KV tiles each query tile needs.
+  // Number of KV tiles each query tile needs; with a window they start with n_pool tiles of pooled rows, and the first token
+  // tile is tile0.
   int n_tiles[NQ];
-  int n_max = 0;
+  int n_max = 0, n_pool = 0, tile0 = 0;
+  auto pooled_rows = [&](int row) {     // pooled rows that query `row` sees
+    const int left = p.pos + row - p.window + 1;
+    return p.pool > 0 && left >= p.pool ? min(left / p.pool, p.pool_rows) : 0;
+  };
+  if constexpr (WIN) {
+    n_pool = (pooled_rows(min(q_row0 + NQ * kAttnBM, p.Sq) - 1) + kAttnBN - 1) / kAttnBN;
+    tile0 = max(0, q_row0 + p.q_offset - p.window + 1) / kAttnBN;
+  }
 #pragma unroll
   for (int t = 0; t < NQ; ++t) {
     const int r0 = q_row0 + t * kAttnBM;
@@ -129,7 +153,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         const int r_last = min(r0 + kAttnBM - 1, p.Sq - 1);
         last_key = min(last_key, r_last + p.q_offset);
       }
-      n = last_key >= 0 ? last_key / kAttnBN + 1 : 0;
+      n = last_key >= 0 ? last_key / kAttnBN + 1 - tile0 + n_pool : 0;
     }
     n_tiles[t] = n;
     n_max = max(n_max, n);
@@ -178,24 +202,34 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       for (int t = 0; t < NQ; ++t) {
         if (n_tiles[t] == 0) continue;
         mbar_arrive_expect_tx(&q_full[t], L::kQBytes);
-        for (int c = 0; c < kChunks; ++c)
-          tma_load_3d(smem + L::kQOff + t * L::kQBytes + c * (kAttnBM * 128), &tmQ, &q_full[t], head * HD + c * 64,
-                      q_row0 + t * kAttnBM, batch);
+        for (int c = 0; c < kChunks; ++c) {
+          uint8_t* dst = smem + L::kQOff + t * L::kQBytes + c * (kAttnBM * 128);
+          if constexpr (WIN) tma_load_4d(dst, &tmQ, &q_full[t], c * 64, head, q_row0 + t * kAttnBM, batch);
+          else tma_load_3d(dst, &tmQ, &q_full[t], head * HD + c * 64, q_row0 + t * kAttnBM, batch);
+        }
       }
       int k_issued = 0, v_issued = 0;
       for (int j = 0; j < n_max; ++j) {
         const int ks = j % KST, vs = j % VST;
         if (!mbar_wait(&k_empty[ks], ((j / KST) & 1) ^ 1, abort_flag, kWaitEmptyTimeout)) break;
         mbar_arrive_expect_tx(&k_full[ks], L::kKVBytes);
-        for (int c = 0; c < kChunks; ++c)
-          tma_load_3d(smem + L::kKOff + ks * L::kKVBytes + c * (kAttnBN * 128), &tmK, &k_full[ks],
-                      kv_head * HD + c * 64, j * kAttnBN, batch);
+        for (int c = 0; c < kChunks; ++c) {
+          uint8_t* dst = smem + L::kKOff + ks * L::kKVBytes + c * (kAttnBN * 128);
+          if constexpr (WIN)
+            tma_load_4d(dst, j < n_pool ? &tmPK : &tmK, &k_full[ks], c * 64, kv_head,
+                        (j < n_pool ? j : j - n_pool + tile0) * kAttnBN, batch);
+          else tma_load_3d(dst, &tmK, &k_full[ks], kv_head * HD + c * 64, j * kAttnBN, batch);
+        }
         k_issued = j + 1;
         if (!mbar_wait(&v_empty[vs], ((j / VST) & 1) ^ 1, abort_flag, kWaitEmptyTimeout)) break;
         mbar_arrive_expect_tx(&v_full[vs], L::kKVBytes);
-        for (int c = 0; c < kChunks; ++c)
-          tma_load_3d(smem + L::kVOff + vs * L::kKVBytes + c * (kAttnBN * 128), &tmV, &v_full[vs],
-                      kv_head * HD + c * 64, j * kAttnBN, batch);
+        for (int c = 0; c < kChunks; ++c) {
+          uint8_t* dst = smem + L::kVOff + vs * L::kKVBytes + c * (kAttnBN * 128);
+          if constexpr (WIN)
+            tma_load_4d(dst, j < n_pool ? &tmPV : &tmV, &v_full[vs], c * 64, kv_head,
+                        (j < n_pool ? j : j - n_pool + tile0) * kAttnBN, batch);
+          else tma_load_3d(dst, &tmV, &v_full[vs], kv_head * HD + c * 64, j * kAttnBN, batch);
+        }
         v_issued = j + 1;
       }
       if (*abort_flag) {
@@ -301,6 +335,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 
     float m_use = -INFINITY;   // the maximum the stored exponentials are relative to (lags the true maximum)
     float l_run = 0.0f;
+    int pool_limit = -1;       // last visible pooled row
+    if constexpr (WIN) {
+      pool_limit = pooled_rows(q_row) - 1;
+      if (p.sink) {
+        m_use = __bfloat162float(p.sink[head]) * 1.4426950408889634f;
+        l_run = 1.0f;
+      }
+    }
     const int key_limit = p.causal ? min(p.Sk - 1, q_row + p.q_offset) : p.Sk - 1;  // last visible key of this row
     bool ok = true;
 #ifdef DPTB_ATTN_PROFILE
@@ -322,11 +364,22 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       mbar_arrive(&s_empty[t]);   // the tensor core may overwrite S_t with the next tile's scores
       ATTN_PROF_MARK(pt2);
 
-      const int key0 = j * kAttnBN;
-      if (key0 + kAttnBN - 1 > key_limit) {   // per-thread; no warp-level operation inside
+      if constexpr (WIN) {
+        const bool pooled = j < n_pool;
+        const int key0 = (pooled ? j : j - n_pool + tile0) * kAttnBN;
+        const int hi = pooled ? pool_limit : key_limit, lo = pooled ? 0 : q_row + p.q_offset - p.window + 1;
+        if (key0 + kAttnBN - 1 > hi || key0 < lo) {
 #pragma unroll
-        for (int i = 0; i < kAttnBN; ++i)
-          if (key0 + i > key_limit) s[i] = 0xff800000u;   // -inf
+          for (int i = 0; i < kAttnBN; ++i)
+            if (key0 + i > hi || key0 + i < lo) s[i] = 0xff800000u;   // -inf
+        }
+      } else {
+        const int key0 = j * kAttnBN;
+        if (key0 + kAttnBN - 1 > key_limit) {   // per-thread; no warp-level operation inside
+#pragma unroll
+          for (int i = 0; i < kAttnBN; ++i)
+            if (key0 + i > key_limit) s[i] = 0xff800000u;   // -inf
+        }
       }
       // three-input maxima: half the instructions of the two-input form
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -433,7 +486,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         // a row without any visible key keeps m_use = -inf (its polynomial exponentials are 2^-127, not 0)
         const bool any_key = l_run > 0.0f && m_use != -INFINITY;
         const float inv = any_key ? 1.0f / l_run : 0.0f;
-        __nv_bfloat16* dst = p.o + ((long long)batch * p.Sq + (live ? q_row : 0)) * p.ldo + (long long)head * HD;
+        const int dv = WIN ? p.dv : HD;
+        __nv_bfloat16* dst = p.o + ((long long)batch * p.Sq + (live ? q_row : 0)) * p.ldo + (long long)head * dv;
 #pragma unroll
         for (int c = 0; c < HD / 32; ++c) {
           uint32_t r[32];
@@ -442,6 +496,23 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           if (live) {
 #pragma unroll
             for (int d = 0; d < 32; d += 8) {
+              if constexpr (WIN) {
+                if (c * 32 + d >= dv) break;
+                if (p.rot) {      // back by the query's position
+                  const float4* cs = reinterpret_cast<const float4*>(p.rot + (long long)(p.pos + q_row) * (dv / 2) +
+                                                                     (c * 32 + d) / 2);
+#pragma unroll
+                  for (int e = 0; e < 8; e += 4) {
+                    const float4 f = cs[e / 4];
+                    const float x0 = __uint_as_float(r[d + e]), y0 = __uint_as_float(r[d + e + 1]);
+                    const float x1 = __uint_as_float(r[d + e + 2]), y1 = __uint_as_float(r[d + e + 3]);
+                    r[d + e] = __float_as_uint(x0 * f.x + y0 * f.y);
+                    r[d + e + 1] = __float_as_uint(y0 * f.x - x0 * f.y);
+                    r[d + e + 2] = __float_as_uint(x1 * f.z + y1 * f.w);
+                    r[d + e + 3] = __float_as_uint(y1 * f.z - x1 * f.w);
+                  }
+                }
+              }
               uint4 u;
               u.x = pack_bf16x2(__uint_as_float(r[d + 0]) * inv, __uint_as_float(r[d + 1]) * inv);
               u.y = pack_bf16x2(__uint_as_float(r[d + 2]) * inv, __uint_as_float(r[d + 3]) * inv);
@@ -507,7 +578,7 @@ static int attn_fwd_launch(const DptbAttnFwdArgs* a, cudaStream_t st) {
   if (rc) return rc;
   rc = encode_tmap_seq(&tmV, a->v, a->Hkv, HD, a->Sk, a->B, a->ldv, kAttnBN, a->kv_batch_rows);
   if (rc) return rc;
-  AttnFwdParams p;
+  AttnFwdParams p = {};
   p.o = static_cast<__nv_bfloat16*>(a->o);
   p.lse = a->lse;
   p.ldo = a->ldo;
@@ -516,10 +587,10 @@ static int attn_fwd_launch(const DptbAttnFwdArgs* a, cudaStream_t st) {
   p.q_offset = a->q_offset;
   p.scale_log2 = a->scale * 1.4426950408889634f;
   p.num_q_blocks = (a->Sq + NQ * kAttnBM - 1) / (NQ * kAttnBM);
-  auto kern = attn_fwd_kernel<HD, NQ, KST, VST, PREC>;
+  auto kern = attn_fwd_kernel<HD, NQ, KST, VST, PREC, false>;
   DPTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal));
   dim3 grid(p.num_q_blocks, a->Hq, a->B);
-  kern<<<grid, kAttnThreads, L::kTotal, st>>>(tmQ, tmK, tmV, p);
+  kern<<<grid, kAttnThreads, L::kTotal, st>>>(tmQ, tmK, tmV, tmK, tmV, p);
   return counted(1, (int)cudaGetLastError());
 }
 
@@ -550,4 +621,66 @@ extern "C" int dptb_attn_fwd(const DptbAttnFwdArgs* a, void* stream) {
   if (a->head_dim == 64) return attn_fwd_launch<64, 2, 2, 2, false>(a, st);
   if (a->head_dim == 128) return attn_fwd_launch<128, 2, 2, 1, false>(a, st);
   return kErrUnsupported;
+}
+
+struct DptbWindowFwdArgs {
+  const void* q;              // [B*S, H * dk]
+  const void* k;              // [B, rows, G * dk]: history, then the step's tokens
+  const void* v;              // [B, rows, G * dv]
+  const void* k_pool;         // [B, pool_rows, G * dk] or null
+  const void* v_pool;
+  const void* sink;
+  const void* rot;
+  void* o;                    // [B*S, H * dv]
+  int B, S, H, G, dk, dv, rows, hist, window, pool, pool_rows, pos;
+  float scale;
+};
+
+static int encode_tmap_heads(CUtensorMap* map, const void* base, int heads, int d, int seq, int batch, int box_rows) {
+  const uint64_t dims[4] = {(uint64_t)d, (uint64_t)heads, (uint64_t)seq, (uint64_t)batch};
+  const uint64_t strides[3] = {(uint64_t)d * 2, (uint64_t)heads * d * 2, (uint64_t)seq * heads * d * 2};
+  const uint32_t box[4] = {64, 1, (uint32_t)box_rows, 1};
+  return encode_tmap_nd_bf16(map, base, 4, dims, strides, box);
+}
+
+template <int HD, int KST, int VST>
+static int window_fwd_launch(const DptbWindowFwdArgs* a, cudaStream_t st) {
+  using L = AttnFwdSmem<HD, 2, KST, VST, true>;
+  CUtensorMap tmQ, tmK, tmV, tmPK, tmPV;
+  int rc = encode_tmap_heads(&tmQ, a->q, a->H, a->dk, a->S, a->B, kAttnBM);
+  if (!rc) rc = encode_tmap_heads(&tmK, a->k, a->G, a->dk, a->rows, a->B, L::kBN);
+  if (!rc) rc = encode_tmap_heads(&tmV, a->v, a->G, a->dv, a->rows, a->B, L::kBN);
+  tmPK = tmK;
+  tmPV = tmV;
+  if (!rc && a->pool > 0) rc = encode_tmap_heads(&tmPK, a->k_pool, a->G, a->dk, a->pool_rows, a->B, L::kBN);
+  if (!rc && a->pool > 0) rc = encode_tmap_heads(&tmPV, a->v_pool, a->G, a->dv, a->pool_rows, a->B, L::kBN);
+  if (rc) return rc;
+  AttnFwdParams p = {};
+  p.o = static_cast<__nv_bfloat16*>(a->o);
+  p.ldo = (long long)a->H * a->dv;
+  p.B = a->B; p.Sq = a->S; p.Sk = a->rows; p.Hq = a->H; p.Hkv = a->G;
+  p.causal = 1;
+  p.q_offset = a->hist;
+  p.scale_log2 = a->scale * 1.4426950408889634f;
+  p.num_q_blocks = (a->S + 2 * kAttnBM - 1) / (2 * kAttnBM);
+  p.window = a->window; p.pool = a->pool; p.pool_rows = a->pool_rows; p.pos = a->pos; p.dv = a->dv;
+  p.sink = static_cast<const __nv_bfloat16*>(a->sink);
+  p.rot = static_cast<const float2*>(a->rot);
+  auto kern = attn_fwd_kernel<HD, 2, KST, VST, true, true>;
+  DPTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal));
+  kern<<<dim3(p.num_q_blocks, a->H, a->B), kAttnThreads, L::kTotal, st>>>(tmQ, tmK, tmV, tmPK, tmPV, p);
+  return counted(1, (int)cudaGetLastError());
+}
+
+// Windowed attention of a long step (S queries at positions pos ... over `hist` earlier tokens and their own).
+extern "C" int dptb_window_attn_fwd(const DptbWindowFwdArgs* a, void* stream) {
+  auto st = static_cast<cudaStream_t>(stream);
+  if (a->B <= 0 || a->S <= 0) return 0;
+  if (a->H <= 0 || a->G <= 0 || a->H % a->G || a->dk <= 0 || a->dv <= 0 || a->H > 65535 || a->B > 65535) return kErrBadShape;
+  if (a->dk % 8 || a->dv % 8 || a->dk > 128 || a->dv > 128) return kErrUnsupported;
+  if (a->window < 1 || a->rows != a->hist + a->S || a->hist < 0 || a->pos < a->hist || a->scale <= 0.0f) return kErrBadShape;
+  if (a->pool > 0 && (!a->k_pool || !a->v_pool || a->pool_rows < 1)) return kErrBadShape;
+  for (const void* q : {a->q, a->k, a->v, a->k_pool, a->v_pool, a->rot, (const void*)a->o})
+    if (reinterpret_cast<uintptr_t>(q) & 15) return kErrBadShape;
+  return a->dk <= 64 && a->dv <= 64 ? window_fwd_launch<64, 4, 4>(a, st) : window_fwd_launch<128, 3, 3>(a, st);
 }

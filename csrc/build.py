@@ -33,8 +33,8 @@ NVCC_FLAGS = [
 ]
 
 COMPONENTS = {
-    "serve": ["gemm", "gemm_nt", "gemm_skinny", "gemm_grouped", "attention_fwd", "latent_attention", "recurrent",
-              "moe_local", "stream_norm", "elementwise"],
+    "serve": ["gemm", "gemm_nt", "gemm_skinny", "gemm_grouped", "attention_fwd", "attention_decode", "latent_attention",
+              "window_attention", "recurrent", "linear_attention", "moe_local", "stream_norm", "branch_norm", "elementwise"],
 }
 
 

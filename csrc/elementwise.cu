@@ -347,24 +347,32 @@ dropout_kernel(const T* __restrict__ x, T* __restrict__ out, long long n, float 
     out[i] = from_f32<T>(uniform01(seed, offset + (unsigned long long)i) >= p ? to_f32(x[i]) * keep_scale : 0.0f);
 }
 
-// SwiGLU gate: out = silu(g) * u, rows x cols with independent leading dimensions.
-template <typename T>
+// Gated unit: out = act(g) * u, rows x cols with independent leading dimensions; act is silu or the tanh form of gelu.
+template <typename T, bool GELU>
+__device__ __forceinline__ float glu_act(float z) {
+  if constexpr (!GELU) return z / (1.0f + __expf(-z));
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  if constexpr (sizeof(T) == 2) return z / (1.0f + __expf(-2.0f * u));    // 1/2 (1 + tanh u) = sigmoid(2 u)
+  else return 0.5f * z * (1.0f + tanhf(u));
+}
+template <typename T, bool GELU>
 __global__ void __launch_bounds__(kEwThreads)
-swiglu_fwd_kernel(const T* __restrict__ g, long long ldg, const T* __restrict__ u, long long ldu, T* __restrict__ out,
-                  long long ldo, long long rows, int cols) {
+glu_fwd_kernel(const T* __restrict__ g, long long ldg, const T* __restrict__ u, long long ldu, T* __restrict__ out,
+               long long ldo, long long rows, int cols) {
+  pdl_wait();
+  pdl_launch_dependents();
   const long long n = rows * cols;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / cols;
     const int c = (int)(i % cols);
-    const float gv = to_f32(g[r * ldg + c]), uv = to_f32(u[r * ldu + c]);
-    out[r * ldo + c] = from_f32<T>(gv / (1.0f + __expf(-gv)) * uv);
+    out[r * ldo + c] = from_f32<T>(glu_act<T, GELU>(to_f32(g[r * ldg + c])) * to_f32(u[r * ldu + c]));
   }
 }
 // 16-byte variants (cols and every leading dimension multiples of 8 elements, 16-byte aligned bases).
-template <typename T>
+template <typename T, bool GELU>
 __global__ void __launch_bounds__(kEwThreads)
-swiglu_fwd_vec8_kernel(const T* __restrict__ g, long long ldg, const T* __restrict__ u, long long ldu,
-                       T* __restrict__ out, long long ldo, long long rows, int cols) {
+glu_fwd_vec8_kernel(const T* __restrict__ g, long long ldg, const T* __restrict__ u, long long ldu,
+                    T* __restrict__ out, long long ldo, long long rows, int cols) {
   pdl_wait();                // (programmatic dependent launch: no-ops in an ordinary launch)
   pdl_launch_dependents();
   const int cv = cols >> 3;
@@ -376,7 +384,7 @@ swiglu_fwd_vec8_kernel(const T* __restrict__ g, long long ldg, const T* __restri
     Vec8<T>::load(g + r * ldg + c, gv);
     Vec8<T>::load(u + r * ldu + c, uv);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) o[j] = gv[j] / (1.0f + __expf(-gv[j])) * uv[j];
+    for (int j = 0; j < 8; ++j) o[j] = glu_act<T, GELU>(gv[j]) * uv[j];
     Vec8<T>::store(out + r * ldo + c, o);
   }
 }
@@ -724,21 +732,28 @@ extern "C" int dptb_dropout(const void* x, void* out, long long n, float p, unsi
                 (dropout_kernel<float><<<ew_grid(n), kEwThreads, 0, st>>>((const float*)x, (float*)out, n, p, seed, offset)));
   return counted(1, (int)cudaGetLastError());
 }
+template <typename T, bool GELU>
+static int launch_glu(const void* g, long long ldg, const void* u, long long ldu, void* out, long long ldo, long long rows,
+                      int cols, cudaStream_t st) {
+  const bool vec = vec8_ok(cols, {ldg, ldu, ldo}, {g, u, out}, sizeof(T));
+  return counted(1, (int)launch_k(vec ? glu_fwd_vec8_kernel<T, GELU> : glu_fwd_kernel<T, GELU>,
+                                  dim3(ew_grid(vec ? rows * (cols >> 3) : rows * cols)), dim3(kEwThreads), 0, st, (const T*)g,
+                                  ldg, (const T*)u, ldu, (T*)out, ldo, rows, cols));
+}
 extern "C" int dptb_swiglu_fwd(const void* g, long long ldg, const void* u, long long ldu, void* out, long long ldo,
                                long long rows, int cols, int dtype, void* stream) {
   if (rows <= 0) return 0;
   auto st = static_cast<cudaStream_t>(stream);
-  if (vec8_ok(cols, {ldg, ldu, ldo}, {g, u, out}, dtype ? 2 : 4)) {
-    const long long nv = rows * (cols >> 3);
-    DPTB_BY_DTYPE(dtype,
-                  (launch_k(swiglu_fwd_vec8_kernel<__nv_bfloat16>, dim3(ew_grid(nv)), dim3(kEwThreads), 0, st, (const __nv_bfloat16*)g, ldg, (const __nv_bfloat16*)u, ldu, (__nv_bfloat16*)out, ldo, rows, cols)),
-                  (swiglu_fwd_vec8_kernel<float><<<ew_grid(nv), kEwThreads, 0, st>>>((const float*)g, ldg, (const float*)u, ldu, (float*)out, ldo, rows, cols)));
-    return counted(1, (int)cudaGetLastError());
-  }
-  DPTB_BY_DTYPE(dtype,
-                (swiglu_fwd_kernel<__nv_bfloat16><<<ew_grid(rows * cols), kEwThreads, 0, st>>>((const __nv_bfloat16*)g, ldg, (const __nv_bfloat16*)u, ldu, (__nv_bfloat16*)out, ldo, rows, cols)),
-                (swiglu_fwd_kernel<float><<<ew_grid(rows * cols), kEwThreads, 0, st>>>((const float*)g, ldg, (const float*)u, ldu, (float*)out, ldo, rows, cols)));
-  return counted(1, (int)cudaGetLastError());
+  return dtype ? launch_glu<__nv_bfloat16, false>(g, ldg, u, ldu, out, ldo, rows, cols, st)
+               : launch_glu<float, false>(g, ldg, u, ldu, out, ldo, rows, cols, st);
+}
+// The same with the tanh form of gelu.
+extern "C" int dptb_geglu_fwd(const void* g, long long ldg, const void* u, long long ldu, void* out, long long ldo,
+                              long long rows, int cols, int dtype, void* stream) {
+  if (rows <= 0) return 0;
+  auto st = static_cast<cudaStream_t>(stream);
+  return dtype ? launch_glu<__nv_bfloat16, true>(g, ldg, u, ldu, out, ldo, rows, cols, st)
+               : launch_glu<float, true>(g, ldg, u, ldu, out, ldo, rows, cols, st);
 }
 extern "C" int dptb_swiglu_bwd(const void* g, long long ldg, const void* u, long long ldu, const void* dout,
                                long long ldo, void* dg, long long lddg, void* du, long long lddu, long long rows,

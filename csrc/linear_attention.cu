@@ -1,0 +1,744 @@
+// Linear attention with a matrix state per head and a decay in front of it:
+//
+//   S_t = diag(a_t) S_{t-1} + k_t v_t^T          S [dk, dv] fp32, zero before the first token
+//   o_t = S_t^T q_t
+//
+// a_t is either one number per key channel and token, a = sigmoid(z)^(1 / tau) with z = W2 r + b from a low-rank projection r
+// of the token (gated linear attention), or one constant per head (lightning attention).  q, k and v are column ranges of one
+// projected row; an activation and the query's scale are applied where they are read.
+//
+//   linear_step      token by token, exact recurrence, any dtype and size: decode steps, short inputs, fp32.  The decay enters
+//                    as a - 1 = expm1(log a), so that long memories do not drift.
+//   decay_kernel     log a for every token and channel of a long input
+//   linear_chunk     bf16, long inputs: pieces of up to 64 tokens as matrix products.  With G the running sum of log a inside
+//                    a piece and G_1 its value at the piece's first token,
+//                        o_i  = (q_i e^{G_i - G_1})^T (e^{G_1} S) + sum_{j <= i} (q_i e^{G_i - G_1}) . (k_j e^{G_1 - G_j}) v_j
+//                        S'   = e^{G_end - G_1} (e^{G_1} S + sum_j (k_j e^{G_1 - G_j}) v_j^T)
+//                    Every operand that carries a decay or the state enters the tensor core as a high and a low bf16 part (16
+//                    mantissa bits), the state itself stays in fp32 registers.  A piece whose decays span more than e^50 is
+//                    cut shorter (down to one token, where the span is zero), so no factor overflows.
+//                    The sequence is cut into segments that run in parallel: pass 1 finds what each segment adds to the state,
+//                    pass 2 folds the segments before its own and computes outputs.
+//   head_norm_gate   rms(o) * w * act(g): the norm over every head (one w for all) or over all heads together
+#include <cuda_bf16.h>
+
+#include "common/host.h"
+#include "common/ptx.cuh"
+#include "common/reduce.cuh"
+
+namespace dptb {
+
+struct LinearParams {
+  const void* p;            // [B*S, ld] projected rows
+  long long ld;
+  int oq, ok, ov, orank;    // column of the queries, keys, values and low-rank decay inputs
+  const void* w2;           // [H * dk, rank] (null: constant decay)
+  const void* b2;           // [H * dk]
+  const float* decay;       // [H, 2]: log a, a - 1
+  float* log_a;             // [B*S, H * dk] (long inputs)
+  float* state;             // [B, H, dk, dv]
+  void* o;                  // [B*S, H * dv]
+  float* ends;              // [B, H, segments + 1, dk, dv]: state a segment adds; the last entry copies the initial state
+  float* totals;            // [B, H, segments, dk]: log decay over a segment
+  int B, S, H, dk, dv, rank, silu, segments, seg_tokens;
+  float q_scale, inv_tau;
+};
+
+__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+// log sigmoid(z)
+__device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
+
+template <typename T>
+__device__ __forceinline__ float low_rank_log_decay(const LinearParams& p, long long row, int hc) {
+  const T* r = static_cast<const T*>(p.p) + row * p.ld + p.orank;
+  const T* w = static_cast<const T*>(p.w2) + (long long)hc * p.rank;
+  float z = to_f32(static_cast<const T*>(p.b2)[hc]);
+  for (int i = 0; i < p.rank; ++i) z = fmaf(to_f32(w[i]), to_f32(r[i]), z);
+  return log_sigmoid_f(z) * p.inv_tau;
+}
+
+// ------------------------------------------------------------------------------------------- token by token
+constexpr int kStepThreads = 256;
+constexpr int kStepCols = 16;       // column groups of V values
+constexpr int kStepRows = 16;       // row groups; a thread holds rows rg, rg + 16, ...
+
+template <typename T, int V, int NR>
+__global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearParams p) {
+  extern __shared__ float step_smem[];
+  const int dk = p.dk, dv = p.dv;
+  float* qs = step_smem;
+  float* ks = qs + dk;
+  float* es = ks + dk;              // a - 1
+  float* red = es + dk;             // [8][kStepCols * V]
+  const int cg = threadIdx.x & (kStepCols - 1), rg = threadIdx.x / kStepCols;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int c0 = (blockIdx.x * kStepCols + cg) * V;
+  const bool live = c0 < dv;
+  // the state was written by an earlier step, several launches ago: it can be fetched before the wait
+  float* state = p.state + ((long long)b * p.H + h) * dk * dv + c0;
+  float S[NR][V];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int r = rg + kStepRows * i;
+#pragma unroll
+    for (int k = 0; k < V; ++k) S[i][k] = 0.0f;
+    if (live && r < dk) {
+      if constexpr (V == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(state + (long long)r * dv);
+        S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
+      } else {
+        S[i][0] = state[(long long)r * dv];
+      }
+    }
+  }
+  const float const_e = p.decay ? p.decay[2 * h + 1] : 0.0f;
+  pdl_wait();
+  pdl_launch_dependents();
+  for (int t = 0; t < p.S; ++t) {
+    const long long row = (long long)b * p.S + t;
+    const T* src = static_cast<const T*>(p.p) + row * p.ld;
+    float v[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      v[k] = live ? to_f32(src[p.ov + h * dv + c0 + k]) : 0.0f;
+      if (p.silu) v[k] = silu_f(v[k]);
+    }
+    for (int c = threadIdx.x; c < dk; c += kStepThreads) {
+      float q = to_f32(src[p.oq + h * dk + c]), k = to_f32(src[p.ok + h * dk + c]);
+      if (p.silu) {
+        q = silu_f(q);
+        k = silu_f(k);
+      }
+      qs[c] = q * p.q_scale;
+      ks[c] = k;
+      es[c] = p.decay ? const_e : expm1f(low_rank_log_decay<T>(p, row, h * dk + c));
+    }
+    __syncthreads();
+    float acc[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) acc[k] = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int r = rg + kStepRows * i;
+      if (r < dk) {
+        const float e = es[r], kk = ks[r], q = qs[r];
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+          S[i][k] += fmaf(e, S[i][k], kk * v[k]);
+          acc[k] = fmaf(q, S[i][k], acc[k]);
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      acc[k] += __shfl_xor_sync(0xffffffffu, acc[k], 16);
+      if (lane < 16) red[warp * (kStepCols * V) + cg * V + k] = acc[k];
+    }
+    __syncthreads();
+    const int out = threadIdx.x;
+    if (out < kStepCols * V && blockIdx.x * kStepCols * V + out < dv) {
+      float s = 0.0f;
+#pragma unroll
+      for (int w = 0; w < kStepThreads / 32; ++w) s += red[w * (kStepCols * V) + out];
+      static_cast<T*>(p.o)[row * p.H * dv + (long long)h * dv + blockIdx.x * kStepCols * V + out] = from_f32<T>(s);
+    }
+  }
+  if (!live) return;
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int r = rg + kStepRows * i;
+    if (r < dk) {
+      if constexpr (V == 4)
+        *reinterpret_cast<float4*>(state + (long long)r * dv) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+      else
+        state[(long long)r * dv] = S[i][0];
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------- decays of a long input
+constexpr int kDecayTokens = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(128) decay_kernel(const LinearParams p) {
+  extern __shared__ float decay_r[];      // [kDecayTokens][rank]
+  const long long row0 = (long long)blockIdx.x * kDecayTokens;
+  const long long rows = (long long)p.B * p.S;
+  const int n = (int)min((long long)kDecayTokens, rows - row0), HK = p.H * p.dk;
+  const int c = blockIdx.y * 128 + threadIdx.x;
+  pdl_wait();
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < kDecayTokens * p.rank; i += 128) {
+    const int t = i / p.rank, r = i % p.rank;
+    decay_r[i] = t < n ? to_f32(static_cast<const T*>(p.p)[(row0 + t) * p.ld + p.orank + r]) : 0.0f;
+  }
+  __syncthreads();
+  if (c >= HK) return;
+  float z[kDecayTokens];
+  const float b = to_f32(static_cast<const T*>(p.b2)[c]);
+#pragma unroll
+  for (int t = 0; t < kDecayTokens; ++t) z[t] = b;
+  const T* w = static_cast<const T*>(p.w2) + (long long)c * p.rank;
+  for (int r = 0; r < p.rank; ++r) {
+    const float wr = to_f32(w[r]);
+#pragma unroll
+    for (int t = 0; t < kDecayTokens; ++t) z[t] = fmaf(wr, decay_r[t * p.rank + r], z[t]);
+  }
+#pragma unroll
+  for (int t = 0; t < kDecayTokens; ++t)
+    if (t < n) p.log_a[(row0 + t) * HK + c] = log_sigmoid_f(z[t]) * p.inv_tau;
+}
+
+// ------------------------------------------------------------------------------------------- pieces of 64 tokens
+constexpr int kLinC = 64;           // tokens of a piece at most
+constexpr int kLinDv = 64;          // value columns of a CTA
+constexpr int kLinThreads = 256;
+constexpr float kLinSpan = 50.0f;   // log decay span of a piece
+constexpr int kVRow = kLinDv + 8;   // padded rows: ldmatrix without bank conflicts
+
+__device__ __forceinline__ void lin_ldm(uint32_t (&r)[4], const __nv_bfloat16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void lin_ldm_t(uint32_t (&r)[4], const __nv_bfloat16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void lin_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
+  hi = __float2bfloat16(v);
+  lo = __float2bfloat16(v - __bfloat162float(hi));
+}
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(a, b);
+  const float2 f = unpack_bf16x2(hi);
+  lo = pack_bf16x2(a - f.x, b - f.y);
+}
+
+template <int DK, bool OUT>
+struct LinSmem {
+  static constexpr int kKRow = DK + 8;
+  static constexpr int kKBytes = kLinC * kKRow * 2;       // one part of the keys (or queries)
+  static constexpr int kVBytes = kLinC * kVRow * 2;
+  static constexpr int kSBytes = DK * kVRow * 2;
+  static constexpr int kK = 0;                            // [2][64][DK + 8] high, low; the scores [2][64][64 + 8] follow
+  static constexpr int kV = kK + 2 * (OUT && kVBytes > kKBytes ? kVBytes : kKBytes);
+  static constexpr int kQ = kV + kVBytes;                 // pass 2 only from here
+  static constexpr int kS = kQ + (OUT ? 2 * kKBytes : 0);
+  static constexpr int kSum = kS + (OUT ? 2 * kSBytes : 0);
+  static constexpr int kParts = kLinThreads / DK;
+  static constexpr int kTotal = kSum + (kParts + 2) * DK * 4;
+  static_assert(kTotal <= 227 * 1024, "linear attention: shared memory budget");
+};
+
+// One CTA: 64 value columns of one head over one segment.  OUT = false: the segment's contribution to the state (pass 1).
+template <int DK, bool OUT>
+__global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const LinearParams p) {
+  using L = LinSmem<DK, OUT>;
+  using bf = __nv_bfloat16;
+  constexpr int KR = L::kKRow;
+  constexpr int MT = DK / 16;                     // 16-row tiles of the state
+  constexpr int MTW = MT > 8 ? MT / 8 : 1;        // ... of a warp
+  constexpr int WN = MT < 8 ? 8 / MT : 1;         // warps side by side along the columns
+  constexpr int NT = 8 / WN;                      // 8-column tiles of a warp
+  constexpr int TP = kLinC / L::kParts;           // tokens a thread prepares
+  extern __shared__ __align__(16) uint8_t lin_smem[];
+  bf* kh = reinterpret_cast<bf*>(lin_smem + L::kK);
+  bf* kl = kh + kLinC * KR;
+  bf* vs = reinterpret_cast<bf*>(lin_smem + L::kV);
+  bf* qh = reinterpret_cast<bf*>(lin_smem + L::kQ);
+  bf* ql = qh + kLinC * KR;
+  bf* sh = reinterpret_cast<bf*>(lin_smem + L::kS);
+  bf* sl = sh + DK * kVRow;
+  bf* ph = reinterpret_cast<bf*>(lin_smem + L::kK);
+  bf* pl = ph + kLinC * kVRow;
+  float* psum = reinterpret_cast<float*>(lin_smem + L::kSum);   // [parts][DK]
+  float* g_in = psum + L::kParts * DK;            // factor on the state before the piece's products
+  float* g_out = g_in + DK;                       // ... and after them
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int seg = blockIdx.x, b = blockIdx.z;
+  const int vt = (p.dv + kLinDv - 1) / kLinDv;
+  const int h = blockIdx.y / vt, v0 = (blockIdx.y % vt) * kLinDv;
+  const int dk = p.dk, dv = p.dv, HK = p.H * dk;
+  const int t_begin = seg * p.seg_tokens, t_end = min(p.S, t_begin + p.seg_tokens);
+  const long long row_b = (long long)b * p.S;
+  const bf* rows = static_cast<const bf*>(p.p) + row_b * p.ld;
+  const float* la_base = p.log_a ? p.log_a + row_b * HK + h * dk : nullptr;
+  pdl_wait();
+  pdl_launch_dependents();
+  const float const_la = p.decay ? p.decay[2 * h] : 0.0f;
+  const int ch = tid % DK, part = tid / DK;       // this thread's channel and share of the tokens while preparing
+  auto log_a = [&](int t) -> float { return ch >= dk ? 0.0f : (la_base ? la_base[(long long)t * HK + ch] : const_la); };
+
+  // the state: warp's row tiles m0 + 128 * i and column tiles n0 + 8 * j
+  const int m0 = (warp / WN) * 16, n0 = (warp % WN) * NT * 8;
+  float S[MTW][NT][4];
+  auto for_state = [&](auto f) {
+#pragma unroll
+    for (int i = 0; i < MTW; ++i)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2)
+          f(i, j, e, m0 + i * 128 + (lane >> 2) + (e >> 1) * 8, n0 + j * 8 + (lane & 3) * 2);
+  };
+  const long long mat = (long long)dk * dv, bh = (long long)b * p.H + h;
+  float* ends = p.ends + bh * (p.segments + 1) * mat;
+  float* totals = p.totals + bh * p.segments * dk;
+  for_state([&](int i, int j, int e, int r, int c) {
+    S[i][j][e] = S[i][j][e + 1] = 0.0f;
+    if ((OUT || seg == 0) && r < dk && v0 + c < dv) {
+      // pass 1 starts the first segment from the state itself and leaves a copy: pass 2 replaces the state
+      const float* src = (OUT && p.segments > 1 ? ends + p.segments * mat : p.state + bh * mat) + (long long)r * dv + v0 + c;
+      const float2 f = *reinterpret_cast<const float2*>(src);
+      S[i][j][e] = f.x;
+      S[i][j][e + 1] = f.y;
+      if (!OUT) *reinterpret_cast<float2*>(ends + p.segments * mat + (long long)r * dv + v0 + c) = f;
+    }
+  });
+  if (OUT && seg > 0) {
+    for_state([&](int i, int j, int e, int r, int c) {
+      if (r < dk && v0 + c < dv) {
+        float2 s = *reinterpret_cast<const float2*>(ends + (long long)r * dv + v0 + c);
+#pragma unroll 4
+        for (int k = 1; k < seg; ++k) {
+          const float2 f = *reinterpret_cast<const float2*>(ends + k * mat + (long long)r * dv + v0 + c);
+          const float d = expm1f(totals[k * dk + r]);
+          s.x += fmaf(d, s.x, f.x);
+          s.y += fmaf(d, s.y, f.y);
+        }
+        S[i][j][e] = s.x;
+        S[i][j][e + 1] = s.y;
+      }
+    });
+  }
+  float total = 0.0f;                             // of channel ch (threads with part == 0)
+  for (int t0 = t_begin; t0 < t_end;) {
+    int n = min(kLinC, t_end - t0);
+    // ---- how much every part decays; a piece whose decays span too much becomes shorter
+    float mine, before = 0.0f, all = 0.0f, first = 0.0f;
+    for (;;) {
+      mine = 0.0f;
+#pragma unroll 8
+      for (int i = 0; i < TP; ++i) {
+        const int t = part * TP + i;
+        if (t < n) mine += log_a(t0 + t);
+      }
+      psum[part * DK + ch] = mine;
+      __syncthreads();
+      before = all = 0.0f;
+#pragma unroll
+      for (int k = 0; k < L::kParts; ++k) {
+        const float s = psum[k * DK + ch];
+        if (k < part) before += s;
+        all += s;
+      }
+      if (!OUT) break;
+      first = log_a(t0);
+      if (!__syncthreads_or(all - first < -kLinSpan) || n == 1) break;
+      n = (n + 3) / 4;
+    }
+    if (part == 0) {
+      g_in[ch] = __expf(OUT ? first : all);
+      g_out[ch] = __expf(all - first);
+      total += all;
+    }
+    // ---- operands: k e^{G_1 - G_j} and q e^{G_i - G_1}; pass 1: k e^{G_end - G_j}
+    float G = before;
+#pragma unroll 8
+    for (int i = 0; i < TP; ++i) {
+      const int t = part * TP + i;
+      float k = 0.0f, q = 0.0f;
+      if (t < n && ch < dk) {
+        G += log_a(t0 + t);
+        const bf* r = rows + (long long)(t0 + t) * p.ld + h * dk + ch;
+        k = __bfloat162float(r[p.ok]);
+        if (p.silu) k = __bfloat162float(__float2bfloat16(silu_f(k)));
+        k *= __expf(OUT ? first - G : all - G);
+        if (OUT) {
+          q = __bfloat162float(r[p.oq]);
+          if (p.silu) q = silu_f(q);
+          q *= p.q_scale * __expf(G - first);
+        }
+      }
+      split_bf16(k, kh[t * KR + ch], kl[t * KR + ch]);
+      if (OUT) split_bf16(q, qh[t * KR + ch], ql[t * KR + ch]);
+    }
+    for (int i = tid; i < kLinC * kLinDv / 8; i += kLinThreads) {
+      const int t = i / (kLinDv / 8), c = i % (kLinDv / 8) * 8;
+      uint4 u = make_uint4(0, 0, 0, 0);
+      if (t < n && v0 + c < dv) u = *reinterpret_cast<const uint4*>(rows + (long long)(t0 + t) * p.ld + p.ov + h * dv + v0 + c);
+      if (p.silu) {
+        uint32_t* w = reinterpret_cast<uint32_t*>(&u);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float2 f = unpack_bf16x2(w[k]);
+          w[k] = pack_bf16x2(silu_f(f.x), silu_f(f.y));
+        }
+      }
+      *reinterpret_cast<uint4*>(vs + t * kVRow + c) = u;
+    }
+    __syncthreads();
+    // ---- the state as the piece's first token sees it
+    for_state([&](int i, int j, int e, int r, int c) {
+      const float g = g_in[r];
+      S[i][j][e] *= g;
+      S[i][j][e + 1] *= g;
+      if (OUT) {
+        uint32_t hi, lo;
+        split_pair(S[i][j][e], S[i][j][e + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(sh + r * kVRow + c) = hi;
+        *reinterpret_cast<uint32_t*>(sl + r * kVRow + c) = lo;
+      }
+    });
+    const int mt = warp & 3, nh = (warp >> 2) * 32;       // this warp's 16 x 32 part of a 64 x 64 product
+    const int a_row = lane & 15, a_col = (lane >> 4) * 8;                          // fragments of A, row-major
+    const int b_row = (lane & 7) + ((lane >> 4) & 1) * 8, b_col = ((lane >> 3) & 1) * 8;   // of B stored [n][k]
+    const int bt_row = (lane & 7) + ((lane >> 3) & 1) * 8, bt_col = ((lane >> 4) & 1) * 8; // of B stored [k][n]
+    float a[4][4];
+    if constexpr (OUT) {
+      // ---- scores of the piece's own tokens
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[j][e] = 0.0f;
+      if (nh <= mt * 16 + 15) {
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          uint32_t ah[4], al[4];
+          lin_ldm(ah, qh + (mt * 16 + a_row) * KR + kk * 16 + a_col);
+          lin_ldm(al, ql + (mt * 16 + a_row) * KR + kk * 16 + a_col);
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            uint32_t bh4[4], bl4[4];
+            lin_ldm(bh4, kh + (nh + j * 16 + b_row) * KR + kk * 16 + b_col);
+            lin_ldm(bl4, kl + (nh + j * 16 + b_row) * KR + kk * 16 + b_col);
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+              lin_mma(a[j * 2 + x], ah, bh4[2 * x], bh4[2 * x + 1]);
+              lin_mma(a[j * 2 + x], ah, bl4[2 * x], bl4[2 * x + 1]);
+              lin_mma(a[j * 2 + x], al, bh4[2 * x], bh4[2 * x + 1]);
+            }
+          }
+        }
+      }
+    }
+    // ---- the state after the piece
+#pragma unroll
+    for (int kk = 0; kk < kLinC / 16; ++kk) {
+      uint32_t vb[NT / 2][4];
+#pragma unroll
+      for (int j = 0; j < NT / 2; ++j) lin_ldm_t(vb[j], vs + (kk * 16 + bt_row) * kVRow + n0 + j * 16 + bt_col);
+#pragma unroll
+      for (int i = 0; i < MTW; ++i) {
+        uint32_t ah[4], al[4];      // transposed: rows are key channels
+        lin_ldm_t(ah, kh + (kk * 16 + b_row) * KR + m0 + i * 128 + b_col);
+        lin_ldm_t(al, kl + (kk * 16 + b_row) * KR + m0 + i * 128 + b_col);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          lin_mma(S[i][j], ah, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
+          lin_mma(S[i][j], al, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
+        }
+      }
+    }
+    if constexpr (OUT) {
+      for_state([&](int i, int j, int e, int r, int c) {
+        const float g = g_out[r];
+        S[i][j][e] *= g;
+        S[i][j][e + 1] *= g;
+      });
+      __syncthreads();          // the keys are done with: the scores take their place
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = nh + j * 8 + (lane & 3) * 2;
+          uint32_t hi, lo;
+          split_pair(c <= r ? a[j][e] : 0.0f, c + 1 <= r ? a[j][e + 1] : 0.0f, hi, lo);
+          *reinterpret_cast<uint32_t*>(ph + r * kVRow + c) = hi;
+          *reinterpret_cast<uint32_t*>(pl + r * kVRow + c) = lo;
+        }
+      __syncthreads();
+      // ---- outputs: own tokens, then everything before the piece
+      float o[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[j][e] = 0.0f;
+      for (int kk = 0; kk <= mt; ++kk) {
+        uint32_t ah[4], al[4];
+        lin_ldm(ah, ph + (mt * 16 + a_row) * kVRow + kk * 16 + a_col);
+        lin_ldm(al, pl + (mt * 16 + a_row) * kVRow + kk * 16 + a_col);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t vb[4];
+          lin_ldm_t(vb, vs + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            lin_mma(o[j * 2 + x], ah, vb[2 * x], vb[2 * x + 1]);
+            lin_mma(o[j * 2 + x], al, vb[2 * x], vb[2 * x + 1]);
+          }
+        }
+      }
+#pragma unroll
+      for (int kk = 0; kk < DK / 16; ++kk) {
+        uint32_t ah[4], al[4];
+        lin_ldm(ah, qh + (mt * 16 + a_row) * KR + kk * 16 + a_col);
+        lin_ldm(al, ql + (mt * 16 + a_row) * KR + kk * 16 + a_col);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t bh4[4], bl4[4];
+          lin_ldm_t(bh4, sh + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
+          lin_ldm_t(bl4, sl + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            lin_mma(o[j * 2 + x], ah, bh4[2 * x], bh4[2 * x + 1]);
+            lin_mma(o[j * 2 + x], ah, bl4[2 * x], bl4[2 * x + 1]);
+            lin_mma(o[j * 2 + x], al, bh4[2 * x], bh4[2 * x + 1]);
+          }
+        }
+      }
+      bf* out = static_cast<bf*>(p.o) + (row_b + t0) * p.H * dv + (long long)h * dv + v0;
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = nh + j * 8 + (lane & 3) * 2;
+          if (r < n && v0 + c < dv)
+            *reinterpret_cast<uint32_t*>(out + (long long)r * p.H * dv + c) = pack_bf16x2(o[j][e], o[j][e + 1]);
+        }
+    }
+    t0 += n;
+    __syncthreads();            // everyone is done with this piece's operands
+  }
+  if (OUT && seg != p.segments - 1) return;
+  float* dst = OUT ? p.state + bh * mat : ends + seg * mat;
+  for_state([&](int i, int j, int e, int r, int c) {
+    if (r < dk && v0 + c < dv)
+      *reinterpret_cast<float2*>(dst + (long long)r * dv + v0 + c) = make_float2(S[i][j][e], S[i][j][e + 1]);
+  });
+  if (!OUT && v0 == 0 && part == 0 && ch < dk) totals[seg * dk + ch] = total;
+}
+
+// ------------------------------------------------------------------------------------------- norm and gate
+struct HeadNormParams {
+  const void* o;            // [rows, groups * n]
+  const void* w;            // [n]
+  const void* g;            // [rows, ldg], same columns as o
+  long long ldg;
+  void* out;                // [rows, groups * n]
+  int groups, n, sigmoid;
+  float eps;
+};
+
+// A warp per (row, group) when n is small, a CTA of 4 warps per (row, group) otherwise.
+template <typename T, int V, bool CTA>
+__global__ void __launch_bounds__(128) head_norm_gate_kernel(const HeadNormParams p, long long units) {
+  __shared__ float scratch[33];
+  constexpr int W = CTA ? 128 : 32;
+  constexpr int kKeep = 4;
+  const int lane = CTA ? threadIdx.x : threadIdx.x & 31;
+  const long long unit = CTA ? blockIdx.x : (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (unit >= units) return;
+  const long long row = unit / p.groups;
+  const int off = (int)(unit % p.groups) * p.n;
+  const T* o = static_cast<const T*>(p.o) + row * p.groups * p.n + off;
+  const T* g = static_cast<const T*>(p.g) + row * p.ldg + off;
+  T* out = static_cast<T*>(p.out) + row * p.groups * p.n + off;
+  auto load = [&](const T* q, float (&x)[V]) {
+    if constexpr (V == 8) Vec8<T>::load(q, x);
+    else x[0] = to_f32(q[0]);
+  };
+  float keep[kKeep][V], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (i * W + lane) * V;
+#pragma unroll
+    for (int k = 0; k < V; ++k) keep[i][k] = 0.0f;
+    if (c < p.n) load(o + c, keep[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i)
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(keep[i][k], keep[i][k], ss);
+  for (int c = (kKeep * W + lane) * V; c < p.n; c += W * V) {
+    float x[V];
+    load(o + c, x);
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(x[k], x[k], ss);
+  }
+  const float inv = 1.0f / sqrtf((CTA ? block_sum(ss, scratch) : warp_sum(ss)) / (float)p.n + p.eps);
+  auto put = [&](int c, const float (&x)[V]) {
+    float w[V], gv[V], y[V];
+    load(static_cast<const T*>(p.w) + c, w);
+    load(g + c, gv);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const float s = 1.0f / (1.0f + expf(-gv[k]));
+      y[k] = x[k] * inv * w[k] * (p.sigmoid ? s : gv[k] * s);
+    }
+    if constexpr (V == 8) Vec8<T>::store(out + c, y);
+    else out[c] = from_f32<T>(y[0]);
+  };
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (i * W + lane) * V;
+    if (c < p.n) put(c, keep[i]);
+  }
+  for (int c = (kKeep * W + lane) * V; c < p.n; c += W * V) {
+    float x[V];
+    load(o + c, x);
+    put(c, x);
+  }
+}
+
+template <typename T, int V>
+static int launch_step(const LinearParams& p, cudaStream_t st) {
+  const dim3 grid((p.dv + kStepCols * V - 1) / (kStepCols * V), p.H, p.B);
+  const size_t smem = (3 * p.dk + 8 * kStepCols * V) * sizeof(float);
+  const int nr = (p.dk + kStepRows - 1) / kStepRows;
+#define DPTB_STEP(NRV) return counted(1, (int)launch_k(linear_step_kernel<T, V, NRV>, grid, dim3(kStepThreads), smem, st, p))
+  if (nr <= 2) DPTB_STEP(2);
+  if (nr <= 4) DPTB_STEP(4);
+  if (nr <= 8) DPTB_STEP(8);
+  if (nr <= 16) DPTB_STEP(16);
+  if (nr <= 32) DPTB_STEP(32);
+#undef DPTB_STEP
+  return kErrUnsupported;
+}
+
+template <int DK>
+static int launch_chunks(const LinearParams& p, cudaStream_t st) {
+  static bool configured = false;
+  if (!configured) {
+    DPTB_CUDA_OK(cudaFuncSetAttribute(linear_chunk_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                      LinSmem<DK, false>::kTotal));
+    DPTB_CUDA_OK(cudaFuncSetAttribute(linear_chunk_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                      LinSmem<DK, true>::kTotal));
+    configured = true;
+  }
+  const unsigned gy = p.H * ((p.dv + kLinDv - 1) / kLinDv);
+  if (p.segments > 1) {
+    const int rc = counted(1, (int)launch_k(linear_chunk_kernel<DK, false>, dim3(p.segments - 1, gy, p.B), dim3(kLinThreads),
+                                            (size_t)LinSmem<DK, false>::kTotal, st, p));
+    if (rc) return rc;
+  }
+  return counted(1, (int)launch_k(linear_chunk_kernel<DK, true>, dim3(p.segments, gy, p.B), dim3(kLinThreads),
+                                  (size_t)LinSmem<DK, true>::kTotal, st, p));
+}
+
+}  // namespace dptb
+
+using namespace dptb;
+
+struct DptbLinearArgs {
+  const void* p; const void* w2; const void* b2; const float* decay; float* log_a; float* state; void* o; float* ws;
+  long long ld, ws_floats;
+  int oq, ok, ov, orank;
+  int B, S, H, dk, dv, rank, silu, f32, chunked, segments;
+  float q_scale, inv_tau;
+};
+
+// Whether long inputs of these sizes run as pieces on the tensor cores.
+extern "C" int dptb_linear_chunkable(int dk, int dv, int f32) { return !f32 && dk <= 256 && dv % 8 == 0 && dk >= 1; }
+
+static int linear_seg_tokens(int S, int segments) { return ((S + segments - 1) / segments + kLinC - 1) / kLinC * kLinC; }
+
+// Segments: enough CTAs to fill the SMs (two fit one up to 64 key channels), four pieces each at least.
+extern "C" int dptb_linear_segments(int B, int S, int H, int dk, int dv) {
+  const int ctas = B * H * ((dv + kLinDv - 1) / kLinDv);
+  int s = (sm_count() * (dk <= 64 ? 2 : 1) + ctas - 1) / ctas;
+  const int by_len = S / (4 * kLinC);
+  if (s > by_len) s = by_len;
+  if (s < 1) s = 1;
+  const int seg = linear_seg_tokens(S, s);
+  return (S + seg - 1) / seg;
+}
+extern "C" long long dptb_linear_ws_floats(int B, int H, int dk, int dv, int segments) {
+  return segments <= 1 ? 0 : (long long)B * H * ((long long)(segments + 1) * dk * dv + (long long)segments * dk);
+}
+
+extern "C" int dptb_linear_attn(const DptbLinearArgs* a, void* stream_v) {
+  auto st = static_cast<cudaStream_t>(stream_v);
+  if (a->B <= 0 || a->S <= 0) return 0;
+  if (a->H <= 0 || a->dk <= 0 || a->dv <= 0 || a->B > 65535 || a->H > 65535) return kErrBadShape;
+  if (!a->decay && (!a->w2 || !a->b2 || a->rank <= 0)) return kErrBadShape;
+  LinearParams p = {};
+  p.p = a->p; p.ld = a->ld; p.oq = a->oq; p.ok = a->ok; p.ov = a->ov; p.orank = a->orank;
+  p.w2 = a->w2; p.b2 = a->b2; p.decay = a->decay; p.state = a->state; p.o = a->o;
+  p.B = a->B; p.S = a->S; p.H = a->H; p.dk = a->dk; p.dv = a->dv; p.rank = a->rank; p.silu = a->silu;
+  p.q_scale = a->q_scale; p.inv_tau = a->inv_tau;
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (!a->chunked) {
+    p.segments = 1;
+    p.seg_tokens = a->S;
+    if (a->dv % 4 == 0 && al16(a->state)) return a->f32 ? launch_step<float, 4>(p, st) : launch_step<__nv_bfloat16, 4>(p, st);
+    return a->f32 ? launch_step<float, 1>(p, st) : launch_step<__nv_bfloat16, 1>(p, st);
+  }
+  if (!dptb_linear_chunkable(a->dk, a->dv, a->f32)) return kErrUnsupported;
+  if (a->ld % 8 || a->ov % 8 || !al16(a->p) || !al16(a->state) || !al16(a->o)) return kErrBadShape;
+  p.segments = a->segments < 1 ? 1 : a->segments;
+  p.seg_tokens = linear_seg_tokens(a->S, p.segments);
+  if ((a->S + p.seg_tokens - 1) / p.seg_tokens != p.segments) return kErrBadShape;
+  if (dptb_linear_ws_floats(a->B, a->H, a->dk, a->dv, p.segments) > a->ws_floats) return kErrTooLarge;
+  if (p.segments > 1 && !al16(a->ws)) return kErrBadShape;
+  p.ends = a->ws;
+  p.totals = a->ws ? a->ws + (long long)a->B * a->H * (p.segments + 1) * a->dk * a->dv : nullptr;
+  if (!a->decay) {
+    if (!a->log_a) return kErrBadShape;
+    p.log_a = a->log_a;
+    const size_t smem = (size_t)kDecayTokens * a->rank * sizeof(float);
+    const long long blocks = ((long long)a->B * a->S + kDecayTokens - 1) / kDecayTokens;
+    if (smem > 48 * 1024 || blocks > 0x7fffffff) return kErrTooLarge;
+    const int rc = counted(1, (int)launch_k(decay_kernel<__nv_bfloat16>, dim3((unsigned)blocks, (a->H * a->dk + 127) / 128),
+                                            dim3(128), smem, st, p));
+    if (rc) return rc;
+  }
+  if (a->dk <= 32) return launch_chunks<32>(p, st);
+  if (a->dk <= 64) return launch_chunks<64>(p, st);
+  if (a->dk <= 128) return launch_chunks<128>(p, st);
+  return launch_chunks<256>(p, st);
+}
+
+struct DptbHeadNormArgs {
+  const void* o; const void* w; const void* g; void* out;
+  long long ldg;
+  int rows, groups, n, sigmoid, f32;
+  float eps;
+};
+
+extern "C" int dptb_head_norm_gate(const DptbHeadNormArgs* a, void* stream_v) {
+  auto st = static_cast<cudaStream_t>(stream_v);
+  if (a->rows <= 0) return 0;
+  if (a->groups <= 0 || a->n <= 0 || a->ldg < (long long)a->groups * a->n) return kErrBadShape;
+  HeadNormParams p;
+  p.o = a->o; p.w = a->w; p.g = a->g; p.ldg = a->ldg; p.out = a->out;
+  p.groups = a->groups; p.n = a->n; p.sigmoid = a->sigmoid; p.eps = a->eps;
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = a->n % 8 == 0 && a->ldg % 8 == 0 && al16(a->o) && al16(a->w) && al16(a->g) && al16(a->out);
+  const long long units = (long long)a->rows * a->groups;
+  const bool cta = a->n > (vec ? 1024 : 128);
+  const long long blocks = cta ? units : (units + 3) / 4;
+  if (blocks > 0x7fffffff) return kErrTooLarge;
+  const dim3 grid((unsigned)blocks);
+#define DPTB_HN(T, V, C) return counted(1, (int)launch_k(head_norm_gate_kernel<T, V, C>, grid, dim3(128), (size_t)0, st, p, units))
+  if (a->f32) {
+    if (vec) { if (cta) DPTB_HN(float, 8, true); DPTB_HN(float, 8, false); }
+    if (cta) DPTB_HN(float, 1, true);
+    DPTB_HN(float, 1, false);
+  }
+  if (vec) { if (cta) DPTB_HN(__nv_bfloat16, 8, true); DPTB_HN(__nv_bfloat16, 8, false); }
+  if (cta) DPTB_HN(__nv_bfloat16, 1, true);
+  DPTB_HN(__nv_bfloat16, 1, false);
+#undef DPTB_HN
+}

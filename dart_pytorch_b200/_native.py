@@ -194,6 +194,7 @@ def _declare(lib: ctypes.CDLL) -> None:
     sig("dptb_rope", P, P, L, I, I, I, I, I, F, I, I, L, L, P, P)
     sig("dptb_dropout", P, P, L, F, ctypes.c_ulonglong, ctypes.c_ulonglong, I, P)
     sig("dptb_swiglu_fwd", P, L, P, L, P, L, L, I, I, P)
+    sig("dptb_geglu_fwd", P, L, P, L, P, L, L, I, I, P)
     sig("dptb_swiglu_bwd", P, L, P, L, P, L, P, L, P, L, L, I, I, P)
     sig("dptb_argmax_rows", P, L, P, L, I, I, P)
     sig("dptb_topk_sample", P, L, P, P, L, I, I, F, I, I, P)

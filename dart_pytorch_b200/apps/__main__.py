@@ -1,7 +1,7 @@
 """Command-line entry points: ``python -m dart_pytorch_b200.apps <command> [options]``
 (reference: the ``bin/`` programs — trainers ``gpt_train``, ``train_char_lm``, ``shakespeare_{gpt,gpt_big,
 transformer_lm,aft,moe}``, ``vit_demo``, ``train_muzero_lm_demo``; runners ``gpt2`` / ``distilgpt2`` / ``pythia`` /
-``gptj`` / ``llama_chat`` / ``famudra`` / ``auto`` with ``--serve``; ``trace_run``; ``rag_chat_server``; ``lc0_demo``; cooperative training ``coop_train_phase0``,
+``gptj`` / ``llama_chat`` / ``famudra`` / ``pozalorn`` / ``auto`` with ``--serve``; ``trace_run``; ``rag_chat_server``; ``lc0_demo``; cooperative training ``coop_train_phase0``,
 ``coop_coordinator``, ``coop_worker``, ``coop_peer``; vector tools ``demo_faiss``, ``bench_faiss``, ``faiss_describe``,
 ``faiss_strip``; and every remaining demo / debug program — ``gpt_demo``, ``lm_demo``, ``aft_demo``, ``aft_bench``,
 ``seq2seq_optim_bench``, ``word2vec_demo``, ``data_loaders_demo``, ``tutorial``, the ``vit_*`` demos,
@@ -184,7 +184,7 @@ def cmd_muzero(args):
 
 
 def cmd_hf_runner(args):
-    """``gpt2`` / ``distilgpt2`` / ``pythia`` / ``gptj`` / ``llama`` / ``famudra`` / ``auto`` runner: one-shot generation or ``--serve``."""
+    """``gpt2`` / ``distilgpt2`` / ``pythia`` / ``gptj`` / ``llama`` / ``famudra`` / ``pozalorn`` / ``auto`` runner: one-shot generation or ``--serve``."""
     from .servers import GenerationService, load_hf_model
     dev = _device(args.device)
     dtype = torch.bfloat16 if (args.bf16 and dev == "cuda") else torch.float32
@@ -384,7 +384,7 @@ def main(argv=None):
         p.add_argument("--device", default="auto")
         p.add_argument("--steps", type=int, default=50)
         p.set_defaults(fn=fn)
-    for fam in ("gpt2", "distilgpt2", "pythia", "gptj", "llama", "famudra", "auto"):
+    for fam in ("gpt2", "distilgpt2", "pythia", "gptj", "llama", "famudra", "pozalorn", "auto"):
         p = sub.add_parser(fam)
         p.add_argument("model_dir")
         p.add_argument("--device", default="auto")

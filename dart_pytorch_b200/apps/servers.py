@@ -32,9 +32,9 @@ from ..coop.http_coop import ServerHandle
 # -------------------------------------------------------------------------------------------- model loading --
 def load_hf_model(family: str, model_dir: str, device=None, dtype=torch.float32, preset: Optional[str] = None):
     """Build and load a causal LM from ``<model_dir>/model.safetensors`` (or a sharded index) and, when present,
-    ``tokenizer.json``.  ``family``: ``gpt2``, ``distilgpt2``, ``pythia``, ``gptj``, ``llama``, ``famudra`` or ``auto`` (the
-    family that ``config.json`` names); ``preset`` picks the size (e.g. ``medium``, ``160m``, ``8b``); without one the size is
-    inferred from the checkpoint's tensor shapes (``famudra``: read from ``config.json``)."""
+    ``tokenizer.json``.  ``family``: ``gpt2``, ``distilgpt2``, ``pythia``, ``gptj``, ``llama``, ``famudra``, ``pozalorn`` or
+    ``auto`` (the family that ``config.json`` names); ``preset`` picks the size (e.g. ``medium``, ``160m``, ``8b``); without one
+    the size is inferred from the checkpoint's tensor shapes (``famudra``, ``pozalorn``: read from ``config.json``)."""
     from ..data.hf_tokenizers import HFBpeTokenizer
     from ..io.hf_loaders import GPT2HFLoader, LlamaHFLoader
     from ..io.hf_loaders_more import GPTJHFLoader, PythiaHFLoader
@@ -75,7 +75,7 @@ def load_hf_model(family: str, model_dir: str, device=None, dtype=torch.float32,
         report = LlamaHFLoader.load_map(model, state)
     elif fam in registry.ARCHITECTURES:
         arch = registry.architecture(fam)
-        model = arch.build(registry.read_config(model_dir), **kw)
+        model = arch.build(registry.read_config(model_dir), state, **kw)
         report = arch.load_map(model, state)
     else:
         raise ValueError(f"unknown model family {family!r}")

@@ -17,4 +17,6 @@ from .vision_language import CLIPVisionConfig, CLIPVisionModel, LlamaVision
 from .lc0 import (Lc0Net, Lc0Reader, Lc0Input, Lc0Weights, Lc0ConvBlock, Lc0SEUnit, Lc0Residual, Lc0Output, START_FEN,
                   startFen)
 from .famudra import Famudra, FamudraConfig, FamudraLayerConfig
+from .hybrid import HybridDecoder
+from .pozalorn import Pozalorn, PozalornConfig, PozalornLayerConfig
 from .registry import ARCHITECTURES, family_of

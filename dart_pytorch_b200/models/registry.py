@@ -15,20 +15,27 @@ HF_MODEL_TYPES = {"gpt2": "gpt2", "gpt_neox": "pythia", "gptj": "gptj", "llama":
 
 @dataclass(frozen=True)
 class Architecture:
-    """A family whose sizes and constants all come from ``config.json``."""
+    """A family whose sizes and constants all come from ``config.json`` and the checkpoint's shapes."""
     family: str
-    build: Callable            # (config dict, **kw) -> model
+    build: Callable            # (config dict, checkpoint or None, **kw) -> model
     load_map: Callable         # (model, state dict) -> LoadReport
 
 
 def _famudra() -> Architecture:
     from ..io.famudra_loader import FamudraLoader
     from .famudra import Famudra, FamudraConfig
-    return Architecture("famudra", lambda config, **kw: Famudra(FamudraConfig.from_json(config, **kw)),
+    return Architecture("famudra", lambda config, state=None, **kw: Famudra(FamudraConfig.from_json(config, **kw)),
                         FamudraLoader.load_map)
 
 
-ARCHITECTURES: Dict[str, Callable[[], Architecture]] = {"famudra": _famudra}
+def _pozalorn() -> Architecture:
+    from ..io.pozalorn_loader import PozalornLoader
+    from .pozalorn import Pozalorn, PozalornConfig
+    return Architecture("pozalorn", lambda config, state=None, **kw: Pozalorn(PozalornConfig.from_json(config, state, **kw)),
+                        PozalornLoader.load_map)
+
+
+ARCHITECTURES: Dict[str, Callable[[], Architecture]] = {"famudra": _famudra, "pozalorn": _pozalorn}
 
 
 def read_config(model_dir: str) -> dict:

@@ -74,8 +74,9 @@ class HybridCache:
     """State of ``batch`` sequences over all layer runs of a model (a layer that runs several times has one state per run).
 
     ``seq_len`` tokens have been processed; ``pos`` is the same number on the device, where the kernels of a captured decode
-    step read it.  Fixed-size state sits in one flat fp32 buffer, so that a reset is one fill.  Latent buffers grow by
-    doubling when a step needs more than their capacity."""
+    step read it.  ``width`` is the size of the row every layer run keeps for a token shift (0: none).  Fixed-size state sits
+    in one flat fp32 buffer, so that a reset is one fill.  What grows with the sequence (latents, pooled blocks, rotary tables)
+    doubles when a step needs more than the capacity."""
 
     def __init__(self, states: List[object], width: int, batch: int, max_len: int, dtype, device, counters: int = 0):
         self.states, self.batch, self.dtype, self.device = states, batch, dtype, torch.device(device)
@@ -113,12 +114,14 @@ class HybridCache:
         """(slices, workspace) of the latent attention kernel; all layers share one workspace."""
         from ..ops import hybrid as Y
         splits, floats = Y.latent_attn_plan(rows, H, R, max_keys, self.dtype == torch.float32)
-        if splits <= 1:
-            return 1, None
+        return (1, None) if splits <= 1 else (splits, self.workspace(rows, floats))
+
+    def workspace(self, rows: int, floats: int) -> torch.Tensor:
+        """fp32 scratch of an attention kernel for steps of ``rows`` rows, shared by all layers."""
         got = self.plan.get(rows)
         if got is None or got.numel() < floats:
             got = self.plan[rows] = torch.empty(floats, dtype=torch.float32, device=self.device)
-        return splits, got
+        return got
 
     def advance(self, n: int) -> None:
         self.seq_len += n

@@ -479,6 +479,16 @@ def swiglu_fwd(g: torch.Tensor, u: torch.Tensor, out: Optional[torch.Tensor] = N
     return out
 
 
+def geglu_fwd(g: torch.Tensor, u: torch.Tensor, out: Optional[torch.Tensor] = None):
+    """``gelu_tanh(g) * u``."""
+    rows, cols = g.shape
+    if out is None:
+        out = torch.empty(rows, cols, dtype=g.dtype, device=g.device)
+    N.check(N.load().dptb_geglu_fwd(g.data_ptr(), _lead(g), u.data_ptr(), _lead(u), out.data_ptr(), _lead(out), rows, cols,
+                                    N.dtype_code(g), N.stream_ptr()), "geglu_fwd")
+    return out
+
+
 def swiglu_bwd(g, u, dout, dg, du):
     lib = N.load()
     rows, cols = g.shape
