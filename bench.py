@@ -40,9 +40,9 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "torch"])
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--batch", type=int, default=MICRO_BATCH)
-    ap.add_argument("--workload", default="gpt2_train", choices=["gpt2_train", "famudra"],
-                    help="famudra: prompt and decode throughput of the hybrid decoder beside Llama at equal size, one GPU")
-    ap.add_argument("--sizes", default="small,medium,large", help="model sizes of the famudra workload")
+    ap.add_argument("--workload", default="gpt2_train", choices=["gpt2_train", "famudra", "pozalorn"],
+                    help="famudra, pozalorn: prompt and decode throughput of a hybrid decoder beside Llama at equal size, one GPU")
+    ap.add_argument("--sizes", default="small,medium,large", help="model sizes of the hybrid workloads")
     return ap.parse_args()
 
 
@@ -308,7 +308,7 @@ def run_reference(args):
     run(args, METRIC, MODEL, SEQ, ClockSampler)
 
 
-def run_famudra(args):
+def run_hybrid(args):
     import torch
     from benchmarks.hybrid_bench import bench_line
     torch.cuda.set_device(0)
@@ -317,8 +317,8 @@ def run_famudra(args):
 
 if __name__ == "__main__":
     a = parse_args()
-    if a.workload == "famudra":
-        run_famudra(a)
+    if a.workload != "gpt2_train":
+        run_hybrid(a)
     elif a.impl == "reference":
         run_reference(a)
     elif a.impl == "torch":

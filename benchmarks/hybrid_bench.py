@@ -1,12 +1,14 @@
-"""Serving throughput of the hybrid decoder (Famudra) beside Llama at equal width and equal active feed-forward size.
+"""Serving throughput of the hybrid decoders (Famudra, Pozalorn) beside Llama at equal width and equal active feed-forward size.
 
     python bench.py --workload famudra             # the same measurement, one JSON line
-    python benchmarks/hybrid_bench.py --sizes small,medium,large
+    python bench.py --workload pozalorn
+    python benchmarks/hybrid_bench.py --family pozalorn --sizes small,medium,large
 
-Random weights, uniform random prompts, bf16, one GPU.  Famudra runs through ``Famudra.step`` (prompts eagerly, decode steps
-as the captured graph); Llama through ``TPLlamaEngine`` with a group of one rank, the package's one-GPU serving path.  Both
-models have the same width, number of layers, vocabulary and context; Llama's SwiGLU width is 2/3 of the feed-forward width a
-Famudra token uses (three matrices against two).  Times are CUDA events; weights and activations exceed L2.
+Random weights, uniform random prompts, bf16, one GPU.  A hybrid decoder runs through its ``step`` (prompts eagerly, decode
+steps as the captured graph); Llama through ``TPLlamaEngine`` with a group of one rank, the package's one-GPU serving path.
+Both models have the same width, number of layers, vocabulary and context.  Llama's SwiGLU width is that of Pozalorn's gated
+feed-forward, or 2/3 of the feed-forward width a Famudra token uses (three matrices against two).  Times are CUDA events;
+weights and activations exceed L2.
 """
 from __future__ import annotations
 
@@ -28,6 +30,13 @@ SIZES = {      # width, layers, heads, head dim, q_rank, kv_rank, recurrence wid
     "large": dict(width=4096, layers=2, heads=32, dim=128, q_rank=1536, kv_rank=512, rec=4096, blocks=16, experts=64, top=6,
                   ff=1408, shared=2816),
 }
+POZALORN_SIZES = {      # width, layers, feed-forward, attention heads of `dim`, window, block; linear attention heads, dim, vdim
+    "small": dict(width=1024, layers=6, ff=2816, heads=16, dim=64, window=1024, pool=16, lin_heads=8, lin_dim=64, lin_vdim=128),
+    "medium": dict(width=2048, layers=6, ff=5504, heads=16, dim=128, window=1024, pool=16, lin_heads=16, lin_dim=64,
+                   lin_vdim=128),
+    "large": dict(width=4096, layers=3, ff=11008, heads=32, dim=128, window=1024, pool=16, lin_heads=32, lin_dim=64,
+                  lin_vdim=128),
+}
 PROMPTS = ((1, 8192), (4, 2048))
 DECODE = ((1, 2048), (32, 2048))
 
@@ -41,6 +50,25 @@ def famudra_config(s) -> dict:
     rec = {"type": "rglru", "mlp": mlp, "mixer": dict(width=s["rec"], blocks=s["blocks"], conv=4)}
     return {"architecture": "Famudra", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6},
             "layers": [rec if i % 2 == 0 else att for i in range(s["layers"])]}
+
+
+def pozalorn_config(s) -> dict:
+    rot = {"base": 500000.0, "dims": s["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    att = dict(heads=s["heads"], kv_heads=max(1, s["heads"] // 4), dim=s["dim"], vdim=s["dim"], rot=rot, scale=s["dim"] ** -0.5)
+    lin = dict(heads=s["lin_heads"], dim=s["lin_dim"], vdim=s["lin_vdim"])
+    mixers = [("gla", dict(lin, tau=16.0)),
+              ("attention", dict(att, mask={"size": s["window"], "pool": s["pool"]})),
+              ("parallel", {"left": dict(att, mask={"size": s["window"]}), "left_scale": 0.5, "right_scale": 0.5,
+                            "right": dict(lin, decay=[0.5 ** (2.0 ** -(8.0 * i / s["lin_heads"])) for i in range(s["lin_heads"])])})]
+    return {"architecture": "Pozalorn", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6},
+            "layers": [{"type": mixers[i % 3][0], "mixer": mixers[i % 3][1], "mlp": {"kind": "dense", "ff": s["ff"]}}
+                       for i in range(s["layers"])]}
+
+
+def families():
+    """name -> (sizes, configuration of a size, Llama's feed-forward width)."""
+    return {"famudra": (SIZES, famudra_config, lambda s: (2 * (s["top"] * s["ff"] + s["shared"]) // 3 + 127) // 128 * 128),
+            "pozalorn": (POZALORN_SIZES, pozalorn_config, lambda s: s["ff"])}
 
 
 def timed(fn, iters: int, warmup: int) -> float:
@@ -57,10 +85,10 @@ def timed(fn, iters: int, warmup: int) -> float:
     return e0.elapsed_time(e1) / iters
 
 
-def measure_famudra(s, steps: int, warmup: int) -> dict:
+def measure_hybrid(family: str, s, steps: int, warmup: int) -> dict:
     from dart_pytorch_b200 import _native
-    from dart_pytorch_b200.models.famudra import Famudra, FamudraConfig
-    model = Famudra(FamudraConfig.from_json(famudra_config(s), device="cuda", dtype=torch.bfloat16, init_std=0.02))
+    from dart_pytorch_b200.models import registry
+    model = registry.architecture(family).build(families()[family][1](s), device="cuda", dtype=torch.bfloat16, init_std=0.02)
     model.eval()
     out = {"params": model.num_scalars(), "prefill": [], "decode": []}
     g = torch.Generator().manual_seed(0)
@@ -87,7 +115,7 @@ def measure_famudra(s, steps: int, warmup: int) -> dict:
     return out
 
 
-def measure_llama(s, steps: int, warmup: int) -> dict:
+def measure_llama(s, ffn: int, steps: int, warmup: int) -> dict:
     import torch.distributed as dist
     from dart_pytorch_b200.models.llama import LlamaConfig
     from dart_pytorch_b200.parallel.tp_llama import TPLlamaEngine
@@ -96,7 +124,6 @@ def measure_llama(s, steps: int, warmup: int) -> dict:
         os.environ.setdefault("MASTER_ADDR", "127.0.0.1")
         os.environ.setdefault("MASTER_PORT", "29577")
         dist.init_process_group("nccl", rank=0, world_size=1, device_id=torch.device("cuda", torch.cuda.current_device()))
-    ffn = (2 * (s["top"] * s["ff"] + s["shared"]) // 3 + 127) // 128 * 128
     heads = s["width"] // s["dim"]
     out = {"ffn_dim": ffn, "prefill": [], "decode": []}
     g = torch.Generator().manual_seed(0)
@@ -122,44 +149,48 @@ def measure_llama(s, steps: int, warmup: int) -> dict:
     return out
 
 
-def measure(sizes, steps: int, warmup: int, llama: bool = True) -> dict:
+def measure(family: str, sizes, steps: int, warmup: int, llama: bool = True) -> dict:
     out = {}
+    table, _, ffn = families()[family]
     for name in sizes:
-        out[name] = {"famudra": measure_famudra(SIZES[name], steps, warmup)}
+        out[name] = {family: measure_hybrid(family, table[name], steps, warmup)}
         torch.cuda.empty_cache()
         if llama:
-            out[name]["llama"] = measure_llama(SIZES[name], steps, warmup)
+            out[name]["llama"] = measure_llama(table[name], ffn(table[name]), steps, warmup)
             torch.cuda.empty_cache()
     return out
 
 
 def bench_line(args, sampler_cls) -> dict:
-    """The line ``bench.py --workload famudra`` prints: decode throughput of the medium size at batch 32 as the value."""
+    """The line ``bench.py --workload <family>`` prints: decode throughput of the medium size at batch 32 as the value."""
+    family, table = args.workload, families()[args.workload][0]
     sampler = sampler_cls(0)
     sampler.start()
     sizes = [s for s in args.sizes.split(",") if s]
     sampler.mark()
-    r = measure(sizes, args.steps, args.warmup)
+    r = measure(family, sizes, args.steps, args.warmup)
     clocks = sampler.stop()
     main = r.get("medium") or r[sizes[0]]
-    dec = main["famudra"]["decode"][-1]
-    return {"metric": "famudra_decode_tokens_per_s", "value": dec["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+    dec = main[family]["decode"][-1]
+    return {"metric": f"{family}_decode_tokens_per_s", "value": dec["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
             "steps": args.steps, "warmup": args.warmup, "ms_per_step": dec["ms"], "higher_is_better": True,
             "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "impl": "ours",
-            "config": {"model": "famudra", "sizes": {k: SIZES[k] for k in sizes},
+            "config": {"model": family, "sizes": {k: table[k] for k in sizes},
                        "cache_policy": "weights and activations exceed the 126 MB L2"},
             "gpu_launches": dec["kernels_per_step"] * args.steps, "clocks": clocks, "sizes": r}
 
 
 def main():
     ap = argparse.ArgumentParser()
+    ap.add_argument("--family", default="famudra", choices=sorted(families()))
     ap.add_argument("--sizes", default="small,medium,large")
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--no-llama", action="store_true")
     args = ap.parse_args()
     torch.cuda.set_device(0)
-    print(json.dumps(measure([s for s in args.sizes.split(",") if s], args.steps, args.warmup, not args.no_llama), indent=1))
+    print(json.dumps(measure(args.family, [s for s in args.sizes.split(",") if s], args.steps, args.warmup, not args.no_llama),
+                     indent=1))
 
 
 if __name__ == "__main__":
