@@ -45,6 +45,7 @@ struct LinearParams {
 };
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+__device__ __forceinline__ float fast_silu_f(float v) { return __fdividef(v, 1.0f + __expf(-v)); }    // bf16 results
 // log sigmoid(z)
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 
@@ -212,37 +213,46 @@ __device__ __forceinline__ void lin_mma(float (&d)[4], const uint32_t (&a)[4], u
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
-  hi = __float2bfloat16(v);
-  lo = __float2bfloat16(v - __bfloat162float(hi));
-}
 __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(a, b);
   const float2 f = unpack_bf16x2(hi);
   lo = pack_bf16x2(a - f.x, b - f.y);
 }
 
+__device__ __forceinline__ void lin_cp16(void* dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void lin_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void lin_cp_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// STAGED: the rows of the next piece (queries, keys, log decays) are copied to shared memory while this one is multiplied;
+// with 256 key channels there is no room for that.
 template <int DK, bool OUT>
 struct LinSmem {
+  static constexpr bool kStaged = DK <= 128;
   static constexpr int kKRow = DK + 8;
   static constexpr int kKBytes = kLinC * kKRow * 2;       // one part of the keys (or queries)
   static constexpr int kVBytes = kLinC * kVRow * 2;
   static constexpr int kSBytes = DK * kVRow * 2;
   static constexpr int kK = 0;                            // [2][64][DK + 8] high, low; the scores [2][64][64 + 8] follow
   static constexpr int kV = kK + 2 * (OUT && kVBytes > kKBytes ? kVBytes : kKBytes);
-  static constexpr int kQ = kV + kVBytes;                 // pass 2 only from here
+  static constexpr int kQ = kV + (kStaged ? 2 : 1) * kVBytes;   // pass 2 only from here
   static constexpr int kS = kQ + (OUT ? 2 * kKBytes : 0);
   static constexpr int kSum = kS + (OUT ? 2 * kSBytes : 0);
-  static constexpr int kParts = kLinThreads / DK;
-  static constexpr int kTotal = kSum + (kParts + 2) * DK * 4;
+  static constexpr int kParts = 2 * kLinThreads / DK;     // a thread prepares two channels of 64 / kParts tokens
+  static constexpr int kRawK = kSum + (kParts + 2) * DK * 4;
+  static constexpr int kRawQ = kRawK + (kStaged ? kLinC * DK * 2 : 0);
+  static constexpr int kRawA = kRawQ + (kStaged && OUT ? kLinC * DK * 2 : 0);
+  static constexpr int kTotal = kRawA + (kStaged ? kLinC * DK * 4 : 0);
   static_assert(kTotal <= 227 * 1024, "linear attention: shared memory budget");
 };
 
 // One CTA: 64 value columns of one head over one segment.  OUT = false: the segment's contribution to the state (pass 1).
 template <int DK, bool OUT>
-__global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const LinearParams p) {
+__global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_kernel(const LinearParams p) {
   using L = LinSmem<DK, OUT>;
   using bf = __nv_bfloat16;
+  constexpr bool STAGED = L::kStaged;
   constexpr int KR = L::kKRow;
   constexpr int MT = DK / 16;                     // 16-row tiles of the state
   constexpr int MTW = MT > 8 ? MT / 8 : 1;        // ... of a warp
@@ -262,6 +272,9 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
   float* psum = reinterpret_cast<float*>(lin_smem + L::kSum);   // [parts][DK]
   float* g_in = psum + L::kParts * DK;            // factor on the state before the piece's products
   float* g_out = g_in + DK;                       // ... and after them
+  bf* raw_k = reinterpret_cast<bf*>(lin_smem + L::kRawK);       // [64][DK]
+  bf* raw_q = reinterpret_cast<bf*>(lin_smem + L::kRawQ);
+  float* raw_a = reinterpret_cast<float*>(lin_smem + L::kRawA);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int seg = blockIdx.x, b = blockIdx.z;
@@ -275,8 +288,45 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
   pdl_wait();
   pdl_launch_dependents();
   const float const_la = p.decay ? p.decay[2 * h] : 0.0f;
-  const int ch = tid % DK, part = tid / DK;       // this thread's channel and share of the tokens while preparing
-  auto log_a = [&](int t) -> float { return ch >= dk ? 0.0f : (la_base ? la_base[(long long)t * HK + ch] : const_la); };
+  const int ch = tid % (DK / 2) * 2, part = tid / (DK / 2);   // this thread's channels and share of the tokens while preparing
+
+  // Values of the piece at t0 into buffer `buf`; with STAGED everything else of it too.
+  auto fetch = [&](int t0, int buf) {
+    bf* v = vs + buf * (kLinC * kVRow);
+    for (int i = tid; i < kLinC * kLinDv / 8; i += kLinThreads) {
+      const int t = i / (kLinDv / 8), c = i % (kLinDv / 8) * 8;
+      const bool ok = t0 + t < t_end && v0 + c < dv;
+      lin_cp16(v + t * kVRow + c, ok ? rows + (long long)(t0 + t) * p.ld + p.ov + h * dv + v0 + c : rows, ok);
+    }
+    if constexpr (STAGED) {
+      for (int i = tid; i < kLinC * DK / 8; i += kLinThreads) {
+        const int t = i / (DK / 8), c = i % (DK / 8) * 8;
+        const bool ok = t0 + t < t_end && c < dk;
+        const bf* r = ok ? rows + (long long)(t0 + t) * p.ld + h * dk + c : rows;
+        lin_cp16(raw_k + t * DK + c, ok ? r + p.ok : r, ok);
+        if (OUT) lin_cp16(raw_q + t * DK + c, ok ? r + p.oq : r, ok);
+      }
+      if (la_base) {
+        for (int i = tid; i < kLinC * DK / 4; i += kLinThreads) {
+          const int t = i / (DK / 4), c = i % (DK / 4) * 4;
+          const bool ok = t0 + t < t_end && c < dk;
+          lin_cp16(raw_a + t * DK + c, ok ? la_base + (long long)(t0 + t) * HK + c : la_base, ok);
+        }
+      }
+    }
+    lin_cp_commit();
+  };
+  // Token t of the piece at t0, channels ch and ch + 1 (channels beyond dk are zero).
+  auto log_a = [&](int t0, int t) -> float2 {
+    if (!la_base) return make_float2(const_la, const_la);
+    if constexpr (STAGED) return *reinterpret_cast<const float2*>(raw_a + t * DK + ch);
+    return ch < dk ? *reinterpret_cast<const float2*>(la_base + (long long)(t0 + t) * HK + ch) : make_float2(0.0f, 0.0f);
+  };
+  auto pair_of = [&](const bf* raw, int col, int t0, int t) -> float2 {
+    if constexpr (STAGED) return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(raw + t * DK + ch));
+    if (ch >= dk) return make_float2(0.0f, 0.0f);
+    return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(rows + (long long)(t0 + t) * p.ld + col + h * dk + ch));
+  };
 
   // the state: warp's row tiles m0 + 128 * i and column tiles n0 + 8 * j
   const int m0 = (warp / WN) * 16, n0 = (warp % WN) * NT * 8;
@@ -320,73 +370,99 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
       }
     });
   }
-  float total = 0.0f;                             // of channel ch (threads with part == 0)
+  float2 total = make_float2(0.0f, 0.0f);         // of this thread's channels (threads with part == 0)
+  int buf = 0;
+  if (t_begin < t_end) fetch(t_begin, 0);
   for (int t0 = t_begin; t0 < t_end;) {
     int n = min(kLinC, t_end - t0);
-    // ---- how much every part decays; a piece whose decays span too much becomes shorter
-    float mine, before = 0.0f, all = 0.0f, first = 0.0f;
-    for (;;) {
-      mine = 0.0f;
-#pragma unroll 8
-      for (int i = 0; i < TP; ++i) {
-        const int t = part * TP + i;
-        if (t < n) mine += log_a(t0 + t);
-      }
-      psum[part * DK + ch] = mine;
-      __syncthreads();
-      before = all = 0.0f;
-#pragma unroll
-      for (int k = 0; k < L::kParts; ++k) {
-        const float s = psum[k * DK + ch];
-        if (k < part) before += s;
-        all += s;
-      }
-      if (!OUT) break;
-      first = log_a(t0);
-      if (!__syncthreads_or(all - first < -kLinSpan) || n == 1) break;
-      n = (n + 3) / 4;
-    }
-    if (part == 0) {
-      g_in[ch] = __expf(OUT ? first : all);
-      g_out[ch] = __expf(all - first);
-      total += all;
-    }
-    // ---- operands: k e^{G_1 - G_j} and q e^{G_i - G_1}; pass 1: k e^{G_end - G_j}
-    float G = before;
-#pragma unroll 8
-    for (int i = 0; i < TP; ++i) {
-      const int t = part * TP + i;
-      float k = 0.0f, q = 0.0f;
-      if (t < n && ch < dk) {
-        G += log_a(t0 + t);
-        const bf* r = rows + (long long)(t0 + t) * p.ld + h * dk + ch;
-        k = __bfloat162float(r[p.ok]);
-        if (p.silu) k = __bfloat162float(__float2bfloat16(silu_f(k)));
-        k *= __expf(OUT ? first - G : all - G);
-        if (OUT) {
-          q = __bfloat162float(r[p.oq]);
-          if (p.silu) q = silu_f(q);
-          q *= p.q_scale * __expf(G - first);
-        }
-      }
-      split_bf16(k, kh[t * KR + ch], kl[t * KR + ch]);
-      if (OUT) split_bf16(q, qh[t * KR + ch], ql[t * KR + ch]);
-    }
-    for (int i = tid; i < kLinC * kLinDv / 8; i += kLinThreads) {
-      const int t = i / (kLinDv / 8), c = i % (kLinDv / 8) * 8;
-      uint4 u = make_uint4(0, 0, 0, 0);
-      if (t < n && v0 + c < dv) u = *reinterpret_cast<const uint4*>(rows + (long long)(t0 + t) * p.ld + p.ov + h * dv + v0 + c);
-      if (p.silu) {
+    lin_cp_wait();
+    if (p.silu) {               // this thread's own copies, in place
+      for (int i = tid; i < kLinC * kLinDv / 8; i += kLinThreads) {
+        uint4* at = reinterpret_cast<uint4*>(vs + buf * (kLinC * kVRow) + i / (kLinDv / 8) * kVRow + i % (kLinDv / 8) * 8);
+        uint4 u = *at;
         uint32_t* w = reinterpret_cast<uint32_t*>(&u);
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
           const float2 f = unpack_bf16x2(w[k]);
-          w[k] = pack_bf16x2(silu_f(f.x), silu_f(f.y));
+          w[k] = pack_bf16x2(fast_silu_f(f.x), fast_silu_f(f.y));
+        }
+        *at = u;
+      }
+    }
+    __syncthreads();            // the piece's rows are there, and everyone is done with the one before
+    const bf* v_now = vs + buf * (kLinC * kVRow);
+    // ---- how much every part decays; a piece whose decays span too much becomes shorter
+    float2 before, all, first = make_float2(0.0f, 0.0f);
+    for (;;) {
+      float2 mine = make_float2(0.0f, 0.0f);
+#pragma unroll
+      for (int i = 0; i < TP; ++i) {
+        const int t = part * TP + i;
+        if (t < n) {
+          const float2 a = log_a(t0, t);
+          mine.x += a.x;
+          mine.y += a.y;
         }
       }
-      *reinterpret_cast<uint4*>(vs + t * kVRow + c) = u;
+      *reinterpret_cast<float2*>(psum + part * DK + ch) = mine;
+      __syncthreads();
+      before = all = make_float2(0.0f, 0.0f);
+#pragma unroll
+      for (int k = 0; k < L::kParts; ++k) {
+        const float2 s = *reinterpret_cast<const float2*>(psum + k * DK + ch);
+        if (k < part) {
+          before.x += s.x;
+          before.y += s.y;
+        }
+        all.x += s.x;
+        all.y += s.y;
+      }
+      if (!OUT) break;
+      first = log_a(t0, 0);
+      if (!__syncthreads_or(fminf(all.x - first.x, all.y - first.y) < -kLinSpan) || n == 1) break;
+      n = (n + 3) / 4;
+    }
+    if (part == 0) {
+      *reinterpret_cast<float2*>(g_in + ch) = OUT ? make_float2(__expf(first.x), __expf(first.y)) :
+                                                    make_float2(__expf(all.x), __expf(all.y));
+      *reinterpret_cast<float2*>(g_out + ch) = make_float2(__expf(all.x - first.x), __expf(all.y - first.y));
+      total.x += all.x;
+      total.y += all.y;
+    }
+    // ---- operands: k e^{G_1 - G_j} and q e^{G_i - G_1}; pass 1: k e^{G_end - G_j}
+    float2 G = before;
+    const float2 ref = OUT ? first : all;
+#pragma unroll
+    for (int i = 0; i < TP; ++i) {
+      const int t = part * TP + i;
+      float2 k = make_float2(0.0f, 0.0f), q = k;
+      if (t < n) {
+        const float2 a = log_a(t0, t);
+        G.x += a.x;
+        G.y += a.y;
+        k = pair_of(raw_k, p.ok, t0, t);
+        if (p.silu) k = unpack_bf16x2(pack_bf16x2(fast_silu_f(k.x), fast_silu_f(k.y)));
+        k.x *= __expf(ref.x - G.x);
+        k.y *= __expf(ref.y - G.y);
+        if (OUT) {
+          q = pair_of(raw_q, p.oq, t0, t);
+          if (p.silu) q = make_float2(fast_silu_f(q.x), fast_silu_f(q.y));
+          q.x *= p.q_scale * __expf(G.x - ref.x);
+          q.y *= p.q_scale * __expf(G.y - ref.y);
+        }
+      }
+      uint32_t hi, lo;
+      split_pair(k.x, k.y, hi, lo);
+      *reinterpret_cast<uint32_t*>(kh + t * KR + ch) = hi;
+      *reinterpret_cast<uint32_t*>(kl + t * KR + ch) = lo;
+      if (OUT) {
+        split_pair(q.x, q.y, hi, lo);
+        *reinterpret_cast<uint32_t*>(qh + t * KR + ch) = hi;
+        *reinterpret_cast<uint32_t*>(ql + t * KR + ch) = lo;
+      }
     }
     __syncthreads();
+    if (STAGED && t0 + n < t_end) fetch(t0 + n, buf ^ 1);
     // ---- the state as the piece's first token sees it
     for_state([&](int i, int j, int e, int r, int c) {
       const float g = g_in[r];
@@ -436,7 +512,7 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
     for (int kk = 0; kk < kLinC / 16; ++kk) {
       uint32_t vb[NT / 2][4];
 #pragma unroll
-      for (int j = 0; j < NT / 2; ++j) lin_ldm_t(vb[j], vs + (kk * 16 + bt_row) * kVRow + n0 + j * 16 + bt_col);
+      for (int j = 0; j < NT / 2; ++j) lin_ldm_t(vb[j], v_now + (kk * 16 + bt_row) * kVRow + n0 + j * 16 + bt_col);
 #pragma unroll
       for (int i = 0; i < MTW; ++i) {
         uint32_t ah[4], al[4];      // transposed: rows are key channels
@@ -480,7 +556,7 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           uint32_t vb[4];
-          lin_ldm_t(vb, vs + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
+          lin_ldm_t(vb, v_now + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
 #pragma unroll
           for (int x = 0; x < 2; ++x) {
             lin_mma(o[j * 2 + x], ah, vb[2 * x], vb[2 * x + 1]);
@@ -517,7 +593,12 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
         }
     }
     t0 += n;
-    __syncthreads();            // everyone is done with this piece's operands
+    if (STAGED) {
+      buf ^= 1;
+    } else if (t0 < t_end) {
+      __syncthreads();
+      fetch(t0, 0);
+    }
   }
   if (OUT && seg != p.segments - 1) return;
   float* dst = OUT ? p.state + bh * mat : ends + seg * mat;
@@ -525,7 +606,7 @@ __global__ void __launch_bounds__(kLinThreads, 1) linear_chunk_kernel(const Line
     if (r < dk && v0 + c < dv)
       *reinterpret_cast<float2*>(dst + (long long)r * dv + v0 + c) = make_float2(S[i][j][e], S[i][j][e + 1]);
   });
-  if (!OUT && v0 == 0 && part == 0 && ch < dk) totals[seg * dk + ch] = total;
+  if (!OUT && v0 == 0 && part == 0 && ch < dk) *reinterpret_cast<float2*>(totals + seg * dk + ch) = total;
 }
 
 // ------------------------------------------------------------------------------------------- norm and gate
@@ -650,14 +731,14 @@ struct DptbLinearArgs {
 };
 
 // Whether long inputs of these sizes run as pieces on the tensor cores.
-extern "C" int dptb_linear_chunkable(int dk, int dv, int f32) { return !f32 && dk <= 256 && dv % 8 == 0 && dk >= 1; }
+extern "C" int dptb_linear_chunkable(int dk, int dv, int f32) { return !f32 && dk <= 256 && dk % 8 == 0 && dv % 8 == 0; }
 
 static int linear_seg_tokens(int S, int segments) { return ((S + segments - 1) / segments + kLinC - 1) / kLinC * kLinC; }
 
-// Segments: enough CTAs to fill the SMs (two fit one up to 64 key channels), four pieces each at least.
+// Segments: as many CTAs as run at once (two fit an SM up to 64 key channels), four pieces each at least.
 extern "C" int dptb_linear_segments(int B, int S, int H, int dk, int dv) {
   const int ctas = B * H * ((dv + kLinDv - 1) / kLinDv);
-  int s = (sm_count() * (dk <= 64 ? 2 : 1) + ctas - 1) / ctas;
+  int s = sm_count() * (dk <= 64 ? 2 : 1) / ctas;
   const int by_len = S / (4 * kLinC);
   if (s > by_len) s = by_len;
   if (s < 1) s = 1;
@@ -686,7 +767,7 @@ extern "C" int dptb_linear_attn(const DptbLinearArgs* a, void* stream_v) {
     return a->f32 ? launch_step<float, 1>(p, st) : launch_step<__nv_bfloat16, 1>(p, st);
   }
   if (!dptb_linear_chunkable(a->dk, a->dv, a->f32)) return kErrUnsupported;
-  if (a->ld % 8 || a->ov % 8 || !al16(a->p) || !al16(a->state) || !al16(a->o)) return kErrBadShape;
+  if (a->ld % 8 || a->oq % 8 || a->ok % 8 || a->ov % 8 || !al16(a->log_a) || !al16(a->p) || !al16(a->state) || !al16(a->o)) return kErrBadShape;
   p.segments = a->segments < 1 ? 1 : a->segments;
   p.seg_tokens = linear_seg_tokens(a->S, p.segments);
   if ((a->S + p.seg_tokens - 1) / p.seg_tokens != p.segments) return kErrBadShape;
