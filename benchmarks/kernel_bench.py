@@ -173,6 +173,101 @@ def build_cases(dev, want=()):
                                 2 * 2 * Bd * Sk * Hkv * hdd, 0.0)
     if on("hybrid"):
         cases.update(build_hybrid_cases(dev))
+    if on("pozalorn"):
+        cases.update(build_pozalorn_cases(dev))
+    return cases
+
+
+def build_pozalorn_cases(dev):
+    """Serving kernels of Pozalorn at the "medium" size of ``hybrid_bench.py``, 4 x 2048 prompt tokens and 32 decode rows after
+    2303 tokens, and (``pozalorn_like_*``) the kernels that play the same part in Llama at that width.  Bytes are what a kernel
+    has to read and write once, products what the equations need (a state update and an output per token, visible keys only)."""
+    from dart_pytorch_b200.nn.mixers import RotaryTable, row_layout
+    from dart_pytorch_b200.ops import decode as Dk
+    from dart_pytorch_b200.ops import mixers as X
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    f32 = dict(device=dev, dtype=torch.float32)
+    D, H, Gk, hd, W, P, LH, dk, dv, ff, layers = 2048, 16, 4, 128, 1024, 16, 16, 64, 128, 5504, 6
+    B, S = 4, 2048
+    M, Bd, at = B * S, 32, 2303
+    rn = lambda *s: torch.randn(*s, **bf)  # noqa: E731
+    cases = {}
+
+    def add(name, fn, nbytes, flops=0.0):
+        cases["pozalorn_" + name] = (fn, nbytes, flops)
+    rot, rot_v = RotaryTable(5e5, hd).rows(4096, dev), RotaryTable(5e5, hd).rows(4096, dev)
+    decays = torch.tensor([0.5 ** (2.0 ** -(8.0 * i / LH)) for i in range(LH)], dtype=torch.float64)
+    decays = torch.stack([decays.log(), decays - 1], 1).float().to(dev)
+    w2, b2 = rn(LH * dk, 16) * 0.1, rn(LH * dk) + 4.0
+    for tag, seqs, rows in (("", B, M), ("dec_", Bd, Bd)):
+        n = rows // seqs
+        # ---- linear attention
+        cols, width = row_layout(q=LH * dk, k=LH * dk, v=LH * dv, g=LH * dv, r=16)
+        p, state = rn(rows, width), torch.zeros(seqs, LH, dk, dv, **f32)
+        nb = 2 * rows * LH * (2 * dk + 2 * dv) + 8 * seqs * LH * dk * dv
+        fl = 4.0 * rows * LH * dk * dv
+        add(tag + "linear_gated", lambda p=p, state=state, seqs=seqs, n=n, cols=cols: X.linear_attn(
+            p, cols, state, seqs, n, LH, dk, dv, w2=w2, b2=b2, tau=16.0, q_scale=dk ** -0.5), nb + 32 * rows, fl)
+        add(tag + "linear_constant", lambda p=p, state=state, seqs=seqs, n=n, cols=cols: X.linear_attn(
+            p, cols, state, seqs, n, LH, dk, dv, decay=decays, silu=True), nb, fl)
+        o, wh, wj = rn(rows, LH * dv), rn(dv), rn(LH * dv)
+        g = p[:, cols["g"]:cols["g"] + LH * dv]
+        add(tag + "norm_gate_head", lambda o=o, g=g: X.head_norm_gate(o, wh, g, 1e-6, "silu"), 6 * rows * LH * dv)
+        add(tag + "norm_gate_joint", lambda o=o, g=g: X.head_norm_gate(o, wj, g, 1e-6, "sigmoid"), 6 * rows * LH * dv)
+        # ---- windowed attention
+        cols, width = row_layout(q=H * hd, k=Gk * hd, v=Gk * hd)
+        p, ring = rn(rows, width), W + 32
+        kr, vr = rn(seqs, ring, Gk * hd), rn(seqs, ring, Gk * hd)
+        kp, vp = rn(seqs, 4096 // P, Gk * hd), rn(seqs, 4096 // P, Gk * hd)
+        kl, vl = (rn(seqs, n, Gk * hd), rn(seqs, n, Gk * hd)) if n > 1 else (None, None)
+        gq, gk = rn(H * hd), rn(Gk * hd)
+        add(tag + "qkv_prep", lambda p=p, seqs=seqs, n=n, kr=kr, vr=vr, kl=kl, vl=vl, cols=cols: X.qkv_prep(
+            p, cols, seqs, n, H, Gk, hd, hd, eps=1e-6, gq=gq, gk=gk, whole=True, rot=rot, rot_v=rot_v, k_ring=kr, v_ring=vr,
+            pos=0 if n > 1 else at, k_lin=kl, v_lin=vl), 4 * rows * width)
+        q, sink = rn(rows, H * hd), rn(H)
+        if n > 1:
+            pairs = sum(min(i + 1, W) + max(0, (i - W + 1) // P) for i in range(n)) * seqs
+            keys = X.WindowKeys(kl, vl, W, pool=P, k_pool=kp, v_pool=vp)
+            add("window_attn_pooled", lambda: X.window_attn_fwd(q0, keys0, B, S, H, Gk, hd, hd, 0, hd ** -0.5, rot=rot_v),
+                4 * rows * (H + Gk) * hd, 4.0 * pairs * H * hd)
+            q0, keys0 = q, keys
+            plain = sum(min(i + 1, W) for i in range(n)) * seqs
+            add("window_attn_sink", lambda: X.window_attn_fwd(q0, X.WindowKeys(keys0.k, keys0.v, W), B, S, H, Gk, hd, hd, 0,
+                                                              hd ** -0.5, sink=sink0), 4 * rows * (H + Gk) * hd, 4.0 * plain * H * hd)
+            sink0 = sink
+            add("pool_blocks", lambda: X.pool_blocks(keys0.k, keys0.v, kp0, vp0, B, pool=P, first=0, count=S // P),
+                4 * rows * Gk * hd)
+            kp0, vp0 = kp, vp
+        else:
+            keys = X.WindowKeys(kr, vr, W, ring=True, pool=P, k_pool=kp, v_pool=vp)
+            count = W + (at - W + 1) // P
+            splits, floats = X.window_decode_plan(Bd, H, Gk, hd, hd, count)
+            ws = torch.empty(max(1, floats), **f32)
+            add("dec_window_attn", lambda: X.window_attn_decode(qd, kd, Bd, 1, H, Gk, hd, hd, at, hd ** -0.5, rot=rot_v,
+                                                                splits=splits, ws=ws), 4 * Bd * count * Gk * hd)
+            qd, kd = q, keys
+        # ---- stream and feed-forward
+        x, m, w, stack = torch.randn(rows, D, **f32), rn(rows, D), rn(D), torch.randn(layers, rows, D, **f32)
+        avg, y, res = rn(4), torch.empty(rows, D, **f32), torch.empty(rows, D, **f32)
+        add(tag + "stream_mixer", lambda x=x, m=m, w=w, y=y, rows=rows: X.branch_norm(
+            x, rows, D, torch.bfloat16, 1e-6, m1=m, m2=m, w=w, x_out=y), rows * D * (4 + 4 + 4 + 2))
+        add(tag + "stream_average", lambda x=x, m=m, w=w, y=y, rows=rows, stack=stack, res=res: X.branch_norm(
+            x, rows, D, torch.bfloat16, 1e-6, m1=m, w=w, stack=stack, n=3, avg=avg, result=res, x_out=y),
+            rows * D * (4 + 2 + 12 + 4 + 4 + 2))
+        gu = rn(rows, 2 * ff)
+        add(tag + "geglu", lambda gu=gu: K.geglu_fwd(gu[:, :ff], gu[:, ff:]), 6 * rows * ff)
+        add("like_" + tag + "swiglu", lambda gu=gu: K.swiglu_fwd(gu[:, :ff], gu[:, ff:]), 6 * rows * ff)
+        add("like_" + tag + "rmsnorm", lambda m=m, w=w: K.rmsnorm_fwd(m, w, 1e-5), 4 * rows * D)
+    # ---- Llama's attention
+    qf, kf, vf, of = rn(M, H * hd), rn(M, Gk * hd), rn(M, Gk * hd), torch.empty(M, H * hd, **bf)
+    add("like_attn_fwd", lambda: A.attn_fwd(qf, kf, vf, B, S, S, H, Gk, hd, True, out=of, need_lse=False),
+        4 * M * (H + Gk) * hd, 2.0 * B * S * S * H * hd)
+    kc, vc, od, qs = rn(Bd, at + 1, Gk * hd), rn(Bd, at + 1, Gk * hd), torch.empty(Bd, H * hd, **bf), rn(Bd, H * hd)
+    add("like_dec_attn", lambda: Dk.attn_decode(qs, kc, vc, Bd, 1, at + 1, H, Gk, hd, at, out=od), 4 * Bd * (at + 1) * Gk * hd)
+    qkv, qkvd = rn(M, (H + 2 * Gk) * hd), rn(Bd, (H + 2 * Gk) * hd)
+    kq, vq = rn(B, S, Gk * hd), rn(B, S, Gk * hd)
+    add("like_rope_append", lambda: Dk.rope_kv_append(qkv, kq, vq, B, S, H, Gk, hd, 0), 4 * M * (H + 2 * Gk) * hd)
+    add("like_dec_rope_append", lambda: Dk.rope_kv_append(qkvd, kc, vc, Bd, 1, H, Gk, hd, at), 4 * Bd * (H + 2 * Gk) * hd)
     return cases
 
 

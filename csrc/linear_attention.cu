@@ -159,11 +159,25 @@ __global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearP
 }
 
 // ------------------------------------------------------------------------------------------- decays of a long input
-constexpr int kDecayTokens = 16;
+constexpr int kDecayTokens = 32;
+
+// log sigmoid(z) with its relative precision also where it is next to 0: log(1 + x) = 2 atanh(x / (2 + x)) by its odd series
+// (x <= 1, so the argument is at most 1/3 and the first term left out is below 2 * 3^-17 / 17).
+__device__ __forceinline__ float log_sigmoid_series_f(float z) {
+  const float x = __expf(-fabsf(z)), s = __fdividef(x, 2.0f + x), s2 = s * s;
+  float r = 1.0f / 15;
+  r = fmaf(r, s2, 1.0f / 13);
+  r = fmaf(r, s2, 1.0f / 11);
+  r = fmaf(r, s2, 1.0f / 9);
+  r = fmaf(r, s2, 1.0f / 7);
+  r = fmaf(r, s2, 1.0f / 5);
+  r = fmaf(r, s2, 1.0f / 3);
+  return fminf(z, 0.0f) - 2.0f * fmaf(r * s2, s, s);
+}
 
 template <typename T>
 __global__ void __launch_bounds__(128) decay_kernel(const LinearParams p) {
-  extern __shared__ float decay_r[];      // [kDecayTokens][rank]
+  extern __shared__ float decay_r[];      // [rank][kDecayTokens]
   const long long row0 = (long long)blockIdx.x * kDecayTokens;
   const long long rows = (long long)p.B * p.S;
   const int n = (int)min((long long)kDecayTokens, rows - row0), HK = p.H * p.dk;
@@ -171,8 +185,8 @@ __global__ void __launch_bounds__(128) decay_kernel(const LinearParams p) {
   pdl_wait();
   pdl_launch_dependents();
   for (int i = threadIdx.x; i < kDecayTokens * p.rank; i += 128) {
-    const int t = i / p.rank, r = i % p.rank;
-    decay_r[i] = t < n ? to_f32(static_cast<const T*>(p.p)[(row0 + t) * p.ld + p.orank + r]) : 0.0f;
+    const int t = i / p.rank, r = i - t * p.rank;
+    decay_r[r * kDecayTokens + t] = t < n ? to_f32(static_cast<const T*>(p.p)[(row0 + t) * p.ld + p.orank + r]) : 0.0f;
   }
   __syncthreads();
   if (c >= HK) return;
@@ -181,22 +195,29 @@ __global__ void __launch_bounds__(128) decay_kernel(const LinearParams p) {
 #pragma unroll
   for (int t = 0; t < kDecayTokens; ++t) z[t] = b;
   const T* w = static_cast<const T*>(p.w2) + (long long)c * p.rank;
+#pragma unroll 4
   for (int r = 0; r < p.rank; ++r) {
     const float wr = to_f32(w[r]);
 #pragma unroll
-    for (int t = 0; t < kDecayTokens; ++t) z[t] = fmaf(wr, decay_r[t * p.rank + r], z[t]);
+    for (int t = 0; t < kDecayTokens; t += 4) {
+      const float4 f = *reinterpret_cast<const float4*>(decay_r + r * kDecayTokens + t);
+      z[t] = fmaf(wr, f.x, z[t]);
+      z[t + 1] = fmaf(wr, f.y, z[t + 1]);
+      z[t + 2] = fmaf(wr, f.z, z[t + 2]);
+      z[t + 3] = fmaf(wr, f.w, z[t + 3]);
+    }
   }
+  float* out = p.log_a + row0 * HK + c;
 #pragma unroll
   for (int t = 0; t < kDecayTokens; ++t)
-    if (t < n) p.log_a[(row0 + t) * HK + c] = log_sigmoid_f(z[t]) * p.inv_tau;
+    if (t < n) out[(long long)t * HK] = log_sigmoid_series_f(z[t]) * p.inv_tau;
 }
 
 // ------------------------------------------------------------------------------------------- pieces of 64 tokens
 constexpr int kLinC = 64;           // tokens of a piece at most
-constexpr int kLinDv = 64;          // value columns of a CTA
-constexpr int kLinThreads = 256;
+constexpr int kLinThreads = 4;      // threads per value column of a CTA
 constexpr float kLinSpan = 50.0f;   // log decay span of a piece
-constexpr int kVRow = kLinDv + 8;   // padded rows: ldmatrix without bank conflicts
+constexpr int kPRow = kLinC + 8;    // padded rows (of the scores): ldmatrix without bank conflicts
 
 __device__ __forceinline__ void lin_ldm(uint32_t (&r)[4], const __nv_bfloat16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -227,19 +248,22 @@ __device__ __forceinline__ void lin_cp_wait() { asm volatile("cp.async.wait_grou
 
 // STAGED: the rows of the next piece (queries, keys, log decays) are copied to shared memory while this one is multiplied;
 // with 256 key channels there is no room for that.
-template <int DK, bool OUT>
+template <int DK, int DV, bool OUT>
 struct LinSmem {
   static constexpr bool kStaged = DK <= 128;
+  static constexpr int kThreads = kLinThreads * DV;
   static constexpr int kKRow = DK + 8;
+  static constexpr int kVRow = DV + 8;
+  static constexpr int kPBytes = kLinC * kPRow * 2;
   static constexpr int kKBytes = kLinC * kKRow * 2;       // one part of the keys (or queries)
   static constexpr int kVBytes = kLinC * kVRow * 2;
   static constexpr int kSBytes = DK * kVRow * 2;
   static constexpr int kK = 0;                            // [2][64][DK + 8] high, low; the scores [2][64][64 + 8] follow
-  static constexpr int kV = kK + 2 * (OUT && kVBytes > kKBytes ? kVBytes : kKBytes);
+  static constexpr int kV = kK + 2 * (OUT && kPBytes > kKBytes ? kPBytes : kKBytes);
   static constexpr int kQ = kV + (kStaged ? 2 : 1) * kVBytes;   // pass 2 only from here
   static constexpr int kS = kQ + (OUT ? 2 * kKBytes : 0);
   static constexpr int kSum = kS + (OUT ? 2 * kSBytes : 0);
-  static constexpr int kParts = 2 * kLinThreads / DK;     // a thread prepares two channels of 64 / kParts tokens
+  static constexpr int kParts = 2 * kThreads / DK;     // a thread prepares two channels of 64 / kParts tokens
   static constexpr int kRawK = kSum + (kParts + 2) * DK * 4;
   static constexpr int kRawQ = kRawK + (kStaged ? kLinC * DK * 2 : 0);
   static constexpr int kRawA = kRawQ + (kStaged && OUT ? kLinC * DK * 2 : 0);
@@ -247,17 +271,20 @@ struct LinSmem {
   static_assert(kTotal <= 227 * 1024, "linear attention: shared memory budget");
 };
 
-// One CTA: 64 value columns of one head over one segment.  OUT = false: the segment's contribution to the state (pass 1).
-template <int DK, bool OUT>
-__global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_kernel(const LinearParams p) {
-  using L = LinSmem<DK, OUT>;
+// One CTA: DV value columns of one head over one segment.  OUT = false: the segment's contribution to the state (pass 1).
+template <int DK, int DV, bool OUT>
+__global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1) linear_chunk_kernel(const LinearParams p) {
+  using L = LinSmem<DK, DV, OUT>;
   using bf = __nv_bfloat16;
   constexpr bool STAGED = L::kStaged;
-  constexpr int KR = L::kKRow;
+  constexpr int KR = L::kKRow, kVRow = L::kVRow, NTHR = L::kThreads;
+  constexpr int WARPS = NTHR / 32;
   constexpr int MT = DK / 16;                     // 16-row tiles of the state
-  constexpr int MTW = MT > 8 ? MT / 8 : 1;        // ... of a warp
-  constexpr int WN = MT < 8 ? 8 / MT : 1;         // warps side by side along the columns
-  constexpr int NT = 8 / WN;                      // 8-column tiles of a warp
+  constexpr int MTW = MT > WARPS ? MT / WARPS : 1;        // ... of a warp
+  constexpr int WN = MT < WARPS ? WARPS / MT : 1; // warps side by side along the columns
+  constexpr int NT = DV / 8 / WN;                 // 8-column tiles of a warp
+  constexpr int NA = 4 * 64 / 8 / WARPS;          // 8-column tiles of a warp's scores (64 x 64 over all warps)
+  static_assert(NT % 2 == 0 && NA % 2 == 0, "fragments of B come in pairs");
   constexpr int TP = kLinC / L::kParts;           // tokens a thread prepares
   extern __shared__ __align__(16) uint8_t lin_smem[];
   bf* kh = reinterpret_cast<bf*>(lin_smem + L::kK);
@@ -268,7 +295,7 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
   bf* sh = reinterpret_cast<bf*>(lin_smem + L::kS);
   bf* sl = sh + DK * kVRow;
   bf* ph = reinterpret_cast<bf*>(lin_smem + L::kK);
-  bf* pl = ph + kLinC * kVRow;
+  bf* pl = ph + kLinC * kPRow;
   float* psum = reinterpret_cast<float*>(lin_smem + L::kSum);   // [parts][DK]
   float* g_in = psum + L::kParts * DK;            // factor on the state before the piece's products
   float* g_out = g_in + DK;                       // ... and after them
@@ -278,8 +305,8 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int seg = blockIdx.x, b = blockIdx.z;
-  const int vt = (p.dv + kLinDv - 1) / kLinDv;
-  const int h = blockIdx.y / vt, v0 = (blockIdx.y % vt) * kLinDv;
+  const int vt = (p.dv + DV - 1) / DV;
+  const int h = blockIdx.y / vt, v0 = (blockIdx.y % vt) * DV;
   const int dk = p.dk, dv = p.dv, HK = p.H * dk;
   const int t_begin = seg * p.seg_tokens, t_end = min(p.S, t_begin + p.seg_tokens);
   const long long row_b = (long long)b * p.S;
@@ -293,13 +320,13 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
   // Values of the piece at t0 into buffer `buf`; with STAGED everything else of it too.
   auto fetch = [&](int t0, int buf) {
     bf* v = vs + buf * (kLinC * kVRow);
-    for (int i = tid; i < kLinC * kLinDv / 8; i += kLinThreads) {
-      const int t = i / (kLinDv / 8), c = i % (kLinDv / 8) * 8;
+    for (int i = tid; i < kLinC * DV / 8; i += NTHR) {
+      const int t = i / (DV / 8), c = i % (DV / 8) * 8;
       const bool ok = t0 + t < t_end && v0 + c < dv;
       lin_cp16(v + t * kVRow + c, ok ? rows + (long long)(t0 + t) * p.ld + p.ov + h * dv + v0 + c : rows, ok);
     }
     if constexpr (STAGED) {
-      for (int i = tid; i < kLinC * DK / 8; i += kLinThreads) {
+      for (int i = tid; i < kLinC * DK / 8; i += NTHR) {
         const int t = i / (DK / 8), c = i % (DK / 8) * 8;
         const bool ok = t0 + t < t_end && c < dk;
         const bf* r = ok ? rows + (long long)(t0 + t) * p.ld + h * dk + c : rows;
@@ -307,7 +334,7 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
         if (OUT) lin_cp16(raw_q + t * DK + c, ok ? r + p.oq : r, ok);
       }
       if (la_base) {
-        for (int i = tid; i < kLinC * DK / 4; i += kLinThreads) {
+        for (int i = tid; i < kLinC * DK / 4; i += NTHR) {
           const int t = i / (DK / 4), c = i % (DK / 4) * 4;
           const bool ok = t0 + t < t_end && c < dk;
           lin_cp16(raw_a + t * DK + c, ok ? la_base + (long long)(t0 + t) * HK + c : la_base, ok);
@@ -338,7 +365,7 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
       for (int j = 0; j < NT; ++j)
 #pragma unroll
         for (int e = 0; e < 4; e += 2)
-          f(i, j, e, m0 + i * 128 + (lane >> 2) + (e >> 1) * 8, n0 + j * 8 + (lane & 3) * 2);
+          f(i, j, e, m0 + i * 16 * WARPS + (lane >> 2) + (e >> 1) * 8, n0 + j * 8 + (lane & 3) * 2);
   };
   const long long mat = (long long)dk * dv, bh = (long long)b * p.H + h;
   float* ends = p.ends + bh * (p.segments + 1) * mat;
@@ -377,8 +404,8 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
     int n = min(kLinC, t_end - t0);
     lin_cp_wait();
     if (p.silu) {               // this thread's own copies, in place
-      for (int i = tid; i < kLinC * kLinDv / 8; i += kLinThreads) {
-        uint4* at = reinterpret_cast<uint4*>(vs + buf * (kLinC * kVRow) + i / (kLinDv / 8) * kVRow + i % (kLinDv / 8) * 8);
+      for (int i = tid; i < kLinC * DV / 8; i += NTHR) {
+        uint4* at = reinterpret_cast<uint4*>(vs + buf * (kLinC * kVRow) + i / (DV / 8) * kVRow + i % (DV / 8) * 8);
         uint4 u = *at;
         uint32_t* w = reinterpret_cast<uint32_t*>(&u);
 #pragma unroll
@@ -475,28 +502,29 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
         *reinterpret_cast<uint32_t*>(sl + r * kVRow + c) = lo;
       }
     });
-    const int mt = warp & 3, nh = (warp >> 2) * 32;       // this warp's 16 x 32 part of a 64 x 64 product
+    const int mt = warp & 3, nh = (warp >> 2) * 32;       // this warp's 16 x 32 part of the outputs
     const int a_row = lane & 15, a_col = (lane >> 4) * 8;                          // fragments of A, row-major
     const int b_row = (lane & 7) + ((lane >> 4) & 1) * 8, b_col = ((lane >> 3) & 1) * 8;   // of B stored [n][k]
     const int bt_row = (lane & 7) + ((lane >> 3) & 1) * 8, bt_col = ((lane >> 4) & 1) * 8; // of B stored [k][n]
-    float a[4][4];
+    const int na = (warp >> 2) * NA * 8;                  // ... and its 16 x 8 NA part of the scores
+    float a[NA][4];
     if constexpr (OUT) {
       // ---- scores of the piece's own tokens
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int j = 0; j < NA; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) a[j][e] = 0.0f;
-      if (nh <= mt * 16 + 15) {
+      if (na <= mt * 16 + 15) {
 #pragma unroll
         for (int kk = 0; kk < DK / 16; ++kk) {
           uint32_t ah[4], al[4];
           lin_ldm(ah, qh + (mt * 16 + a_row) * KR + kk * 16 + a_col);
           lin_ldm(al, ql + (mt * 16 + a_row) * KR + kk * 16 + a_col);
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
+          for (int j = 0; j < NA / 2; ++j) {
             uint32_t bh4[4], bl4[4];
-            lin_ldm(bh4, kh + (nh + j * 16 + b_row) * KR + kk * 16 + b_col);
-            lin_ldm(bl4, kl + (nh + j * 16 + b_row) * KR + kk * 16 + b_col);
+            lin_ldm(bh4, kh + (na + j * 16 + b_row) * KR + kk * 16 + b_col);
+            lin_ldm(bl4, kl + (na + j * 16 + b_row) * KR + kk * 16 + b_col);
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
               lin_mma(a[j * 2 + x], ah, bh4[2 * x], bh4[2 * x + 1]);
@@ -516,8 +544,8 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
 #pragma unroll
       for (int i = 0; i < MTW; ++i) {
         uint32_t ah[4], al[4];      // transposed: rows are key channels
-        lin_ldm_t(ah, kh + (kk * 16 + b_row) * KR + m0 + i * 128 + b_col);
-        lin_ldm_t(al, kl + (kk * 16 + b_row) * KR + m0 + i * 128 + b_col);
+        lin_ldm_t(ah, kh + (kk * 16 + b_row) * KR + m0 + i * 16 * WARPS + b_col);
+        lin_ldm_t(al, kl + (kk * 16 + b_row) * KR + m0 + i * 16 * WARPS + b_col);
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
           lin_mma(S[i][j], ah, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
@@ -533,14 +561,14 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
       });
       __syncthreads();          // the keys are done with: the scores take their place
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int j = 0; j < NA; ++j)
 #pragma unroll
         for (int e = 0; e < 4; e += 2) {
-          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = nh + j * 8 + (lane & 3) * 2;
+          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = na + j * 8 + (lane & 3) * 2;
           uint32_t hi, lo;
           split_pair(c <= r ? a[j][e] : 0.0f, c + 1 <= r ? a[j][e + 1] : 0.0f, hi, lo);
-          *reinterpret_cast<uint32_t*>(ph + r * kVRow + c) = hi;
-          *reinterpret_cast<uint32_t*>(pl + r * kVRow + c) = lo;
+          *reinterpret_cast<uint32_t*>(ph + r * kPRow + c) = hi;
+          *reinterpret_cast<uint32_t*>(pl + r * kPRow + c) = lo;
         }
       __syncthreads();
       // ---- outputs: own tokens, then everything before the piece
@@ -551,8 +579,8 @@ __global__ void __launch_bounds__(kLinThreads, DK <= 64 ? 2 : 1) linear_chunk_ke
         for (int e = 0; e < 4; ++e) o[j][e] = 0.0f;
       for (int kk = 0; kk <= mt; ++kk) {
         uint32_t ah[4], al[4];
-        lin_ldm(ah, ph + (mt * 16 + a_row) * kVRow + kk * 16 + a_col);
-        lin_ldm(al, pl + (mt * 16 + a_row) * kVRow + kk * 16 + a_col);
+        lin_ldm(ah, ph + (mt * 16 + a_row) * kPRow + kk * 16 + a_col);
+        lin_ldm(al, pl + (mt * 16 + a_row) * kPRow + kk * 16 + a_col);
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           uint32_t vb[4];
@@ -620,22 +648,21 @@ struct HeadNormParams {
   float eps;
 };
 
-// A warp per (row, group) when n is small, a CTA of 4 warps per (row, group) otherwise.
-template <typename T, int V, bool CTA>
-__global__ void __launch_bounds__(128) head_norm_gate_kernel(const HeadNormParams p, long long units) {
+// LG lanes per (row, group); 128: a whole CTA.
+template <typename T, int V, int LG>
+__global__ void __launch_bounds__(128) head_norm_gate_kernel(const HeadNormParams p, int units) {
   __shared__ float scratch[33];
-  constexpr int W = CTA ? 128 : 32;
-  constexpr int kKeep = 4;
-  const int lane = CTA ? threadIdx.x : threadIdx.x & 31;
-  const long long unit = CTA ? blockIdx.x : (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  constexpr bool FAST = sizeof(T) == 2;
+  constexpr int kKeep = LG == 128 ? 4 : 2;
+  const int lane = threadIdx.x % LG;
+  const int wanted = blockIdx.x * (128 / LG) + threadIdx.x / LG, unit = min(wanted, units - 1);
   pdl_wait();
   pdl_launch_dependents();
-  if (unit >= units) return;
-  const long long row = unit / p.groups;
-  const int off = (int)(unit % p.groups) * p.n;
-  const T* o = static_cast<const T*>(p.o) + row * p.groups * p.n + off;
+  const int row = unit / p.groups, off = (unit - row * p.groups) * p.n;
+  const long long at = (long long)row * p.groups * p.n + off;
+  const T* o = static_cast<const T*>(p.o) + at;
   const T* g = static_cast<const T*>(p.g) + row * p.ldg + off;
-  T* out = static_cast<T*>(p.out) + row * p.groups * p.n + off;
+  T* out = static_cast<T*>(p.out) + at;
   auto load = [&](const T* q, float (&x)[V]) {
     if constexpr (V == 8) Vec8<T>::load(q, x);
     else x[0] = to_f32(q[0]);
@@ -643,7 +670,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const HeadNormParam
   float keep[kKeep][V], ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < kKeep; ++i) {
-    const int c = (i * W + lane) * V;
+    const int c = (i * LG + lane) * V;
 #pragma unroll
     for (int k = 0; k < V; ++k) keep[i][k] = 0.0f;
     if (c < p.n) load(o + c, keep[i]);
@@ -652,20 +679,27 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const HeadNormParam
   for (int i = 0; i < kKeep; ++i)
 #pragma unroll
     for (int k = 0; k < V; ++k) ss = fmaf(keep[i][k], keep[i][k], ss);
-  for (int c = (kKeep * W + lane) * V; c < p.n; c += W * V) {
+  for (int c = (kKeep * LG + lane) * V; c < p.n; c += LG * V) {
     float x[V];
     load(o + c, x);
 #pragma unroll
     for (int k = 0; k < V; ++k) ss = fmaf(x[k], x[k], ss);
   }
-  const float inv = 1.0f / sqrtf((CTA ? block_sum(ss, scratch) : warp_sum(ss)) / (float)p.n + p.eps);
+  if constexpr (LG == 128) {
+    ss = block_sum(ss, scratch);
+  } else {
+#pragma unroll
+    for (int x = LG / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+  }
+  const float inv = 1.0f / sqrtf(ss / (float)p.n + p.eps);
+  if (wanted >= units) return;
   auto put = [&](int c, const float (&x)[V]) {
     float w[V], gv[V], y[V];
     load(static_cast<const T*>(p.w) + c, w);
     load(g + c, gv);
 #pragma unroll
     for (int k = 0; k < V; ++k) {
-      const float s = 1.0f / (1.0f + expf(-gv[k]));
+      const float s = FAST ? __fdividef(1.0f, 1.0f + __expf(-gv[k])) : 1.0f / (1.0f + expf(-gv[k]));
       y[k] = x[k] * inv * w[k] * (p.sigmoid ? s : gv[k] * s);
     }
     if constexpr (V == 8) Vec8<T>::store(out + c, y);
@@ -673,14 +707,25 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const HeadNormParam
   };
 #pragma unroll
   for (int i = 0; i < kKeep; ++i) {
-    const int c = (i * W + lane) * V;
+    const int c = (i * LG + lane) * V;
     if (c < p.n) put(c, keep[i]);
   }
-  for (int c = (kKeep * W + lane) * V; c < p.n; c += W * V) {
+  for (int c = (kKeep * LG + lane) * V; c < p.n; c += LG * V) {
     float x[V];
     load(o + c, x);
     put(c, x);
   }
+}
+template <typename T, int V>
+static int launch_head_norm(const HeadNormParams& p, int units, cudaStream_t st) {
+  const int vecs = (p.n + V - 1) / V;
+#define DPTB_HN(LG) return counted(1, (int)launch_k(head_norm_gate_kernel<T, V, LG>, dim3((units + 128 / LG - 1) / (128 / LG)), \
+                                                    dim3(128), (size_t)0, st, p, units))
+  if (vecs <= 8) DPTB_HN(8);
+  if (vecs <= 16) DPTB_HN(16);
+  if (vecs <= 96) DPTB_HN(32);
+  DPTB_HN(128);
+#undef DPTB_HN
 }
 
 template <typename T, int V>
@@ -698,24 +743,24 @@ static int launch_step(const LinearParams& p, cudaStream_t st) {
   return kErrUnsupported;
 }
 
-template <int DK>
+template <int DK, int DV>
 static int launch_chunks(const LinearParams& p, cudaStream_t st) {
+  using L1 = LinSmem<DK, DV, false>;
+  using L2 = LinSmem<DK, DV, true>;
   static bool configured = false;
   if (!configured) {
-    DPTB_CUDA_OK(cudaFuncSetAttribute(linear_chunk_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                      LinSmem<DK, false>::kTotal));
-    DPTB_CUDA_OK(cudaFuncSetAttribute(linear_chunk_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                      LinSmem<DK, true>::kTotal));
+    DPTB_CUDA_OK(cudaFuncSetAttribute(linear_chunk_kernel<DK, DV, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, L1::kTotal));
+    DPTB_CUDA_OK(cudaFuncSetAttribute(linear_chunk_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, L2::kTotal));
     configured = true;
   }
-  const unsigned gy = p.H * ((p.dv + kLinDv - 1) / kLinDv);
+  const unsigned gy = p.H * ((p.dv + DV - 1) / DV);
   if (p.segments > 1) {
-    const int rc = counted(1, (int)launch_k(linear_chunk_kernel<DK, false>, dim3(p.segments - 1, gy, p.B), dim3(kLinThreads),
-                                            (size_t)LinSmem<DK, false>::kTotal, st, p));
+    const int rc = counted(1, (int)launch_k(linear_chunk_kernel<DK, DV, false>, dim3(p.segments - 1, gy, p.B), dim3(L1::kThreads),
+                                            (size_t)L1::kTotal, st, p));
     if (rc) return rc;
   }
-  return counted(1, (int)launch_k(linear_chunk_kernel<DK, true>, dim3(p.segments, gy, p.B), dim3(kLinThreads),
-                                  (size_t)LinSmem<DK, true>::kTotal, st, p));
+  return counted(1, (int)launch_k(linear_chunk_kernel<DK, DV, true>, dim3(p.segments, gy, p.B), dim3(L2::kThreads),
+                                  (size_t)L2::kTotal, st, p));
 }
 
 }  // namespace dptb
@@ -735,10 +780,13 @@ extern "C" int dptb_linear_chunkable(int dk, int dv, int f32) { return !f32 && d
 
 static int linear_seg_tokens(int S, int segments) { return ((S + segments - 1) / segments + kLinC - 1) / kLinC * kLinC; }
 
-// Segments: as many CTAs as run at once (two fit an SM up to 64 key channels), four pieces each at least.
+// Value columns of a CTA.
+static int linear_dv(int dk, int dv) { return dk <= 64 && dv > 64 ? 128 : 64; }
+
+// Segments: as many CTAs as run at once (two of 64 columns fit an SM up to 64 key channels), four pieces each at least.
 extern "C" int dptb_linear_segments(int B, int S, int H, int dk, int dv) {
-  const int ctas = B * H * ((dv + kLinDv - 1) / kLinDv);
-  int s = sm_count() * (dk <= 64 ? 2 : 1) / ctas;
+  const int cols = linear_dv(dk, dv), ctas = B * H * ((dv + cols - 1) / cols);
+  int s = sm_count() * (dk <= 64 && cols == 64 ? 2 : 1) / ctas;
   const int by_len = S / (4 * kLinC);
   if (s > by_len) s = by_len;
   if (s < 1) s = 1;
@@ -785,10 +833,11 @@ extern "C" int dptb_linear_attn(const DptbLinearArgs* a, void* stream_v) {
                                             dim3(128), smem, st, p));
     if (rc) return rc;
   }
-  if (a->dk <= 32) return launch_chunks<32>(p, st);
-  if (a->dk <= 64) return launch_chunks<64>(p, st);
-  if (a->dk <= 128) return launch_chunks<128>(p, st);
-  return launch_chunks<256>(p, st);
+  const bool wide = linear_dv(a->dk, a->dv) == 128;
+  if (a->dk <= 32) return wide ? launch_chunks<32, 128>(p, st) : launch_chunks<32, 64>(p, st);
+  if (a->dk <= 64) return wide ? launch_chunks<64, 128>(p, st) : launch_chunks<64, 64>(p, st);
+  if (a->dk <= 128) return launch_chunks<128, 64>(p, st);
+  return launch_chunks<256, 64>(p, st);
 }
 
 struct DptbHeadNormArgs {
@@ -808,18 +857,7 @@ extern "C" int dptb_head_norm_gate(const DptbHeadNormArgs* a, void* stream_v) {
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   const bool vec = a->n % 8 == 0 && a->ldg % 8 == 0 && al16(a->o) && al16(a->w) && al16(a->g) && al16(a->out);
   const long long units = (long long)a->rows * a->groups;
-  const bool cta = a->n > (vec ? 1024 : 128);
-  const long long blocks = cta ? units : (units + 3) / 4;
-  if (blocks > 0x7fffffff) return kErrTooLarge;
-  const dim3 grid((unsigned)blocks);
-#define DPTB_HN(T, V, C) return counted(1, (int)launch_k(head_norm_gate_kernel<T, V, C>, grid, dim3(128), (size_t)0, st, p, units))
-  if (a->f32) {
-    if (vec) { if (cta) DPTB_HN(float, 8, true); DPTB_HN(float, 8, false); }
-    if (cta) DPTB_HN(float, 1, true);
-    DPTB_HN(float, 1, false);
-  }
-  if (vec) { if (cta) DPTB_HN(__nv_bfloat16, 8, true); DPTB_HN(__nv_bfloat16, 8, false); }
-  if (cta) DPTB_HN(__nv_bfloat16, 1, true);
-  DPTB_HN(__nv_bfloat16, 1, false);
-#undef DPTB_HN
+  if (units > 0x7fffffff - 128) return kErrTooLarge;
+  if (a->f32) return vec ? launch_head_norm<float, 8>(p, (int)units, st) : launch_head_norm<float, 1>(p, (int)units, st);
+  return vec ? launch_head_norm<__nv_bfloat16, 8>(p, (int)units, st) : launch_head_norm<__nv_bfloat16, 1>(p, (int)units, st);
 }

@@ -82,9 +82,10 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prep_kernel(const PrepParams
   for (int c = tid * V; c < nq + nk; c += kPrepThreads * V) {
     float v[V];
     load(c < nq ? src + p.oq + c : src + p.ok + c - nq, v);
+    if constexpr (V == 8) Vec8<float>::store(x + c, v);
+    else x[c] = v[0];
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      x[c + e] = v[e];
       if (c < nq) sq = fmaf(v[e], v[e], sq);
       else sk = fmaf(v[e], v[e], sk);
     }
@@ -111,19 +112,22 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prep_kernel(const PrepParams
   const bool keep = s >= p.S - p.ring;        // an earlier token's row would be overwritten by this step's own
   const long long lin = (long long)b * p.lin_rows + p.hist + s;
   const float2* rot = p.rot + (long long)pos * (p.rot_dims / 2);
-  auto normed = [&](int c) {                  // feature c of [q | k] after the norm
-    if (!p.gq) return x[c];
+  auto normed = [&](int c, int d, float (&v)[V]) {     // features c ... of [q | k] (feature d of their head) after the norm
+    if constexpr (V == 8) Vec8<float>::load(x + c, v);
+    else v[0] = x[c];
+    if (!p.gq) return;
     const bool is_k = c >= nq;
-    const int h = c / p.dk;
-    const int g = p.whole ? (is_k ? c - nq : c) : c - h * p.dk;
-    return x[c] * inv[h] * to_f32(static_cast<const T*>(is_k ? p.gk : p.gq)[g]);
+    float g[V];
+    load(static_cast<const T*>(is_k ? p.gk : p.gq) + (p.whole ? (is_k ? c - nq : c) : d), g);
+    const float s = inv[(c - d) / p.dk];
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] *= s * g[e];
   };
   for (int c = tid * V; c < nq + nk; c += kPrepThreads * V) {
     float v[V];
     const int d = c % p.dk;
+    normed(c, d, v);
     if constexpr (V == 8) {
-#pragma unroll
-      for (int e = 0; e < V; ++e) v[e] = normed(c + e);
 #pragma unroll
       for (int e = 0; e < V; e += 2) {
         if (d + e < p.rot_dims) {
@@ -133,13 +137,12 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prep_kernel(const PrepParams
           v[e + 1] = o * cs.x + a * cs.y;
         }
       }
-    } else {
-      v[0] = normed(c);
-      if (d < p.rot_dims) {
-        const float2 cs = rot[d / 2];
-        const float o = normed(d & 1 ? c - 1 : c + 1);
-        v[0] = d & 1 ? v[0] * cs.x + o * cs.y : v[0] * cs.x - o * cs.y;
-      }
+    } else if (d < p.rot_dims) {
+      float o[V];
+      const int step = d & 1 ? -1 : 1;
+      normed(c + step, d + step, o);
+      const float2 cs = rot[d / 2];
+      v[0] = d & 1 ? v[0] * cs.x + o[0] * cs.y : v[0] * cs.x - o[0] * cs.y;
     }
     if (c < nq) {
       store(static_cast<T*>(p.q) + (long long)row * nq + c, v);
@@ -358,7 +361,7 @@ extern "C" int dptb_qkv_prep(const DptbPrepArgs* a, void* stream_v) {
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   bool vec = a->dk % 8 == 0 && a->dv % 8 == 0 && a->ld % 8 == 0 && a->oq % 8 == 0 && a->ok % 8 == 0 && a->ov % 8 == 0;
   for (const void* q : {a->p, (const void*)a->q, (const void*)a->k_ring, (const void*)a->v_ring, (const void*)a->k_lin,
-                        (const void*)a->v_lin})
+                        (const void*)a->v_lin, a->gq, a->gk})
     vec = vec && al16(q);
   const size_t smem = ((size_t)(a->H + a->G) * (a->dk + 1)) * sizeof(float);
   if (smem > 200 * 1024) return kErrTooLarge;
