@@ -9,13 +9,13 @@
 //
 //   linear_step      token by token, exact recurrence, any dtype and size: decode steps, short inputs, fp32.  The decay enters
 //                    as a - 1 = expm1(log a), so that long memories do not drift.
-//   decay_kernel     log a for every token and channel of a long input
+//   decay_kernel     running sums of log2 a over blocks of 64 tokens of a long input
 //   linear_chunk     bf16, long inputs: pieces of up to 64 tokens as matrix products.  With G the running sum of log a inside
 //                    a piece and G_1 its value at the piece's first token,
 //                        o_i  = (q_i e^{G_i - G_1})^T (e^{G_1} S) + sum_{j <= i} (q_i e^{G_i - G_1}) . (k_j e^{G_1 - G_j}) v_j
 //                        S'   = e^{G_end - G_1} (e^{G_1} S + sum_j (k_j e^{G_1 - G_j}) v_j^T)
 //                    Every operand that carries a decay or the state enters the tensor core as a high and a low bf16 part (16
-//                    mantissa bits), the state itself stays in fp32 registers.  A piece whose decays span more than e^50 is
+//                    mantissa bits), the state itself stays in fp32 registers.  A piece whose decays span more than 2^72 is
 //                    cut shorter (down to one token, where the span is zero), so no factor overflows.
 //                    The sequence is cut into segments that run in parallel: pass 1 finds what each segment adds to the state,
 //                    pass 2 folds the segments before its own and computes outputs.
@@ -35,11 +35,11 @@ struct LinearParams {
   const void* w2;           // [H * dk, rank] (null: constant decay)
   const void* b2;           // [H * dk]
   const float* decay;       // [H, 2]: log a, a - 1
-  float* log_a;             // [B*S, H * dk] (long inputs)
+  float* log_a;             // [B*S, H * dk] (long inputs): log2 a summed from the start of the token's block of 64
   float* state;             // [B, H, dk, dv]
   void* o;                  // [B*S, H * dv]
   float* ends;              // [B, H, segments + 1, dk, dv]: state a segment adds; the last entry copies the initial state
-  float* totals;            // [B, H, segments, dk]: log decay over a segment
+  float* totals;            // [B, H, segments, dk]: decay over a segment, minus one
   int B, S, H, dk, dv, rank, silu, segments, seg_tokens;
   float q_scale, inv_tau;
 };
@@ -159,64 +159,80 @@ __global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearP
 }
 
 // ------------------------------------------------------------------------------------------- decays of a long input
-constexpr int kDecayTokens = 32;
+constexpr int kLinC = 64;           // tokens of a block
+constexpr float kLog2e = 1.4426950408889634f;
 
-// log sigmoid(z) with its relative precision also where it is next to 0: log(1 + x) = 2 atanh(x / (2 + x)) by its odd series
-// (x <= 1, so the argument is at most 1/3 and the first term left out is below 2 * 3^-17 / 17).
-__device__ __forceinline__ float log_sigmoid_series_f(float z) {
-  const float x = __expf(-fabsf(z)), s = __fdividef(x, 2.0f + x), s2 = s * s;
-  float r = 1.0f / 15;
-  r = fmaf(r, s2, 1.0f / 13);
-  r = fmaf(r, s2, 1.0f / 11);
-  r = fmaf(r, s2, 1.0f / 9);
-  r = fmaf(r, s2, 1.0f / 7);
-  r = fmaf(r, s2, 1.0f / 5);
-  r = fmaf(r, s2, 1.0f / 3);
-  return fminf(z, 0.0f) - 2.0f * fmaf(r * s2, s, s);
+__device__ __forceinline__ float lin_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 
+// log sigmoid(z) with its relative precision also where it is next to 0: log(1 + x) = 2 atanh(x / (2 + x)) by its odd series
+// (x <= 1, so the argument is at most 1/3 and the first term left out is below 2 * 3^-13 / 13).
+__device__ __forceinline__ float log_sigmoid_series_f(float z) {
+  const float x = lin_exp2(-fabsf(z) * kLog2e);
+  float s;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(s) : "f"(2.0f + x));
+  s *= x;
+  const float s2 = s * s;
+  float r = 2.0f / 11;
+  r = fmaf(r, s2, 2.0f / 9);
+  r = fmaf(r, s2, 2.0f / 7);
+  r = fmaf(r, s2, 2.0f / 5);
+  r = fmaf(r, s2, 2.0f / 3);
+  r = fmaf(r, s2, 2.0f);
+  return fmaf(-r, s, fminf(z, 0.0f));
+}
+
+// A thread per key channel and block of 64 tokens.
 template <typename T>
 __global__ void __launch_bounds__(128) decay_kernel(const LinearParams p) {
-  extern __shared__ float decay_r[];      // [rank][kDecayTokens]
-  const long long row0 = (long long)blockIdx.x * kDecayTokens;
-  const long long rows = (long long)p.B * p.S;
-  const int n = (int)min((long long)kDecayTokens, rows - row0), HK = p.H * p.dk;
+  extern __shared__ float decay_r[];      // [rank][kLinC]
+  constexpr int kHalf = kLinC / 2;
+  const int t0 = blockIdx.x * kLinC, n = min(kLinC, p.S - t0), HK = p.H * p.dk;
+  const long long row0 = (long long)blockIdx.z * p.S + t0;
   const int c = blockIdx.y * 128 + threadIdx.x;
   pdl_wait();
   pdl_launch_dependents();
-  for (int i = threadIdx.x; i < kDecayTokens * p.rank; i += 128) {
-    const int t = i / p.rank, r = i - t * p.rank;
-    decay_r[r * kDecayTokens + t] = t < n ? to_f32(static_cast<const T*>(p.p)[(row0 + t) * p.ld + p.orank + r]) : 0.0f;
+  for (int i = threadIdx.x; i < kLinC * p.rank; i += 128) {
+    const int t = i % kLinC, r = i / kLinC;
+    decay_r[i] = t < n ? to_f32(static_cast<const T*>(p.p)[(row0 + t) * p.ld + p.orank + r]) : 0.0f;
   }
   __syncthreads();
   if (c >= HK) return;
-  float z[kDecayTokens];
-  const float b = to_f32(static_cast<const T*>(p.b2)[c]);
-#pragma unroll
-  for (int t = 0; t < kDecayTokens; ++t) z[t] = b;
+  const float b = to_f32(static_cast<const T*>(p.b2)[c]), scale = p.inv_tau * kLog2e;
   const T* w = static_cast<const T*>(p.w2) + (long long)c * p.rank;
-#pragma unroll 4
-  for (int r = 0; r < p.rank; ++r) {
-    const float wr = to_f32(w[r]);
+  float* out = p.log_a + row0 * HK + c;
+  float G = 0.0f;
 #pragma unroll
-    for (int t = 0; t < kDecayTokens; t += 4) {
-      const float4 f = *reinterpret_cast<const float4*>(decay_r + r * kDecayTokens + t);
-      z[t] = fmaf(wr, f.x, z[t]);
-      z[t + 1] = fmaf(wr, f.y, z[t + 1]);
-      z[t + 2] = fmaf(wr, f.z, z[t + 2]);
-      z[t + 3] = fmaf(wr, f.w, z[t + 3]);
+  for (int half = 0; half < 2; ++half) {
+    f32x2 z[kHalf / 2];
+#pragma unroll
+    for (int t = 0; t < kHalf / 2; ++t) z[t] = f2_splat(b);
+#pragma unroll 4
+    for (int r = 0; r < p.rank; ++r) {
+      const f32x2 wr = f2_splat(to_f32(w[r]));
+#pragma unroll
+      for (int t = 0; t < kHalf / 2; t += 2) {
+        const float4 f = *reinterpret_cast<const float4*>(decay_r + r * kLinC + half * kHalf + 2 * t);
+        z[t] = f2_fma(wr, f2_pack(f.x, f.y), z[t]);
+        z[t + 1] = f2_fma(wr, f2_pack(f.z, f.w), z[t + 1]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < kHalf; ++t) {
+      float lo, hi;
+      f2_unpack(z[t / 2], lo, hi);
+      G += log_sigmoid_series_f(t & 1 ? hi : lo) * scale;
+      if (half * kHalf + t < n) out[(long long)(half * kHalf + t) * HK] = G;
     }
   }
-  float* out = p.log_a + row0 * HK + c;
-#pragma unroll
-  for (int t = 0; t < kDecayTokens; ++t)
-    if (t < n) out[(long long)t * HK] = log_sigmoid_series_f(z[t]) * p.inv_tau;
 }
 
 // ------------------------------------------------------------------------------------------- pieces of 64 tokens
-constexpr int kLinC = 64;           // tokens of a piece at most
 constexpr int kLinThreads = 4;      // threads per value column of a CTA
-constexpr float kLinSpan = 50.0f;   // log decay span of a piece
+constexpr float kLinSpan = 72.0f;   // log2 decay span of a piece
 constexpr int kPRow = kLinC + 8;    // padded rows (of the scores): ldmatrix without bank conflicts
 
 __device__ __forceinline__ void lin_ldm(uint32_t (&r)[4], const __nv_bfloat16* p) {
@@ -262,9 +278,9 @@ struct LinSmem {
   static constexpr int kV = kK + 2 * (OUT && kPBytes > kKBytes ? kPBytes : kKBytes);
   static constexpr int kQ = kV + (kStaged ? 2 : 1) * kVBytes;   // pass 2 only from here
   static constexpr int kS = kQ + (OUT ? 2 * kKBytes : 0);
-  static constexpr int kSum = kS + (OUT ? 2 * kSBytes : 0);
+  static constexpr int kGate = kS + (OUT ? 2 * kSBytes : 0);
   static constexpr int kParts = 2 * kThreads / DK;     // a thread prepares two channels of 64 / kParts tokens
-  static constexpr int kRawK = kSum + (kParts + 2) * DK * 4;
+  static constexpr int kRawK = kGate + 2 * DK * 4;
   static constexpr int kRawQ = kRawK + (kStaged ? kLinC * DK * 2 : 0);
   static constexpr int kRawA = kRawQ + (kStaged && OUT ? kLinC * DK * 2 : 0);
   static constexpr int kTotal = kRawA + (kStaged ? kLinC * DK * 4 : 0);
@@ -296,8 +312,7 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
   bf* sl = sh + DK * kVRow;
   bf* ph = reinterpret_cast<bf*>(lin_smem + L::kK);
   bf* pl = ph + kLinC * kPRow;
-  float* psum = reinterpret_cast<float*>(lin_smem + L::kSum);   // [parts][DK]
-  float* g_in = psum + L::kParts * DK;            // factor on the state before the piece's products
+  float* g_in = reinterpret_cast<float*>(lin_smem + L::kGate);  // factor on the state before the piece's products
   float* g_out = g_in + DK;                       // ... and after them
   bf* raw_k = reinterpret_cast<bf*>(lin_smem + L::kRawK);       // [64][DK]
   bf* raw_q = reinterpret_cast<bf*>(lin_smem + L::kRawQ);
@@ -314,7 +329,8 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
   const float* la_base = p.log_a ? p.log_a + row_b * HK + h * dk : nullptr;
   pdl_wait();
   pdl_launch_dependents();
-  const float const_la = p.decay ? p.decay[2 * h] : 0.0f;
+  const float const_la = p.decay ? p.decay[2 * h] * kLog2e : 0.0f;
+  const float q_shift = OUT ? log2f(p.q_scale) : 0.0f;
   const int ch = tid % (DK / 2) * 2, part = tid / (DK / 2);   // this thread's channels and share of the tokens while preparing
 
   // Values of the piece at t0 into buffer `buf`; with STAGED everything else of it too.
@@ -343,9 +359,10 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
     }
     lin_cp_commit();
   };
-  // Token t of the piece at t0, channels ch and ch + 1 (channels beyond dk are zero).
-  auto log_a = [&](int t0, int t) -> float2 {
-    if (!la_base) return make_float2(const_la, const_la);
+  // Token t of the piece at t0, channels ch and ch + 1 (channels beyond dk are zero): the decay summed from the block's start
+  // (constant decays: from the piece's).
+  auto decayed = [&](int t0, int t) -> float2 {
+    if (!la_base) return make_float2((t + 1) * const_la, (t + 1) * const_la);
     if constexpr (STAGED) return *reinterpret_cast<const float2*>(raw_a + t * DK + ch);
     return ch < dk ? *reinterpret_cast<const float2*>(la_base + (long long)(t0 + t) * HK + ch) : make_float2(0.0f, 0.0f);
   };
@@ -388,7 +405,7 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
 #pragma unroll 4
         for (int k = 1; k < seg; ++k) {
           const float2 f = *reinterpret_cast<const float2*>(ends + k * mat + (long long)r * dv + v0 + c);
-          const float d = expm1f(totals[k * dk + r]);
+          const float d = totals[k * dk + r];
           s.x += fmaf(d, s.x, f.x);
           s.y += fmaf(d, s.y, f.y);
         }
@@ -398,10 +415,11 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
     });
   }
   float2 total = make_float2(0.0f, 0.0f);         // of this thread's channels (threads with part == 0)
+  float2 base = make_float2(0.0f, 0.0f);          // decay of the block before the piece
   int buf = 0;
   if (t_begin < t_end) fetch(t_begin, 0);
   for (int t0 = t_begin; t0 < t_end;) {
-    int n = min(kLinC, t_end - t0);
+    int n = min(kLinC - t0 % kLinC, t_end - t0);  // pieces do not cross blocks
     lin_cp_wait();
     if (p.silu) {               // this thread's own copies, in place
       for (int i = tid; i < kLinC * DV / 8; i += NTHR) {
@@ -418,64 +436,47 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
     }
     __syncthreads();            // the piece's rows are there, and everyone is done with the one before
     const bf* v_now = vs + buf * (kLinC * kVRow);
-    // ---- how much every part decays; a piece whose decays span too much becomes shorter
-    float2 before, all, first = make_float2(0.0f, 0.0f);
-    for (;;) {
-      float2 mine = make_float2(0.0f, 0.0f);
-#pragma unroll
-      for (int i = 0; i < TP; ++i) {
-        const int t = part * TP + i;
-        if (t < n) {
-          const float2 a = log_a(t0, t);
-          mine.x += a.x;
-          mine.y += a.y;
-        }
+    // ---- a piece whose decays span too much becomes shorter
+    auto decay_to = [&](int t) {
+      float2 g = decayed(t0, t);
+      if (la_base) {
+        g.x -= base.x;
+        g.y -= base.y;
       }
-      *reinterpret_cast<float2*>(psum + part * DK + ch) = mine;
-      __syncthreads();
-      before = all = make_float2(0.0f, 0.0f);
-#pragma unroll
-      for (int k = 0; k < L::kParts; ++k) {
-        const float2 s = *reinterpret_cast<const float2*>(psum + k * DK + ch);
-        if (k < part) {
-          before.x += s.x;
-          before.y += s.y;
-        }
-        all.x += s.x;
-        all.y += s.y;
+      return g;
+    };
+    float2 all = decay_to(n - 1), first = make_float2(0.0f, 0.0f);
+    if constexpr (OUT) {
+      first = decay_to(0);
+      while (__syncthreads_or(fminf(all.x - first.x, all.y - first.y) < -kLinSpan) && n > 1) {
+        n = (n + 3) / 4;
+        all = decay_to(n - 1);
       }
-      if (!OUT) break;
-      first = log_a(t0, 0);
-      if (!__syncthreads_or(fminf(all.x - first.x, all.y - first.y) < -kLinSpan) || n == 1) break;
-      n = (n + 3) / 4;
     }
     if (part == 0) {
-      *reinterpret_cast<float2*>(g_in + ch) = OUT ? make_float2(__expf(first.x), __expf(first.y)) :
-                                                    make_float2(__expf(all.x), __expf(all.y));
-      *reinterpret_cast<float2*>(g_out + ch) = make_float2(__expf(all.x - first.x), __expf(all.y - first.y));
+      *reinterpret_cast<float2*>(g_in + ch) = OUT ? make_float2(lin_exp2(first.x), lin_exp2(first.y)) :
+                                                    make_float2(lin_exp2(all.x), lin_exp2(all.y));
+      *reinterpret_cast<float2*>(g_out + ch) = make_float2(lin_exp2(all.x - first.x), lin_exp2(all.y - first.y));
       total.x += all.x;
       total.y += all.y;
     }
     // ---- operands: k e^{G_1 - G_j} and q e^{G_i - G_1}; pass 1: k e^{G_end - G_j}
-    float2 G = before;
-    const float2 ref = OUT ? first : all;
+    const float2 ref = OUT ? first : all, ref_q = make_float2(first.x - q_shift, first.y - q_shift);
 #pragma unroll
     for (int i = 0; i < TP; ++i) {
       const int t = part * TP + i;
       float2 k = make_float2(0.0f, 0.0f), q = k;
       if (t < n) {
-        const float2 a = log_a(t0, t);
-        G.x += a.x;
-        G.y += a.y;
+        const float2 G = decay_to(t);
         k = pair_of(raw_k, p.ok, t0, t);
         if (p.silu) k = unpack_bf16x2(pack_bf16x2(fast_silu_f(k.x), fast_silu_f(k.y)));
-        k.x *= __expf(ref.x - G.x);
-        k.y *= __expf(ref.y - G.y);
+        k.x *= lin_exp2(ref.x - G.x);
+        k.y *= lin_exp2(ref.y - G.y);
         if (OUT) {
           q = pair_of(raw_q, p.oq, t0, t);
           if (p.silu) q = make_float2(fast_silu_f(q.x), fast_silu_f(q.y));
-          q.x *= p.q_scale * __expf(G.x - ref.x);
-          q.y *= p.q_scale * __expf(G.y - ref.y);
+          q.x *= lin_exp2(G.x - ref_q.x);
+          q.y *= lin_exp2(G.y - ref_q.y);
         }
       }
       uint32_t hi, lo;
@@ -502,7 +503,8 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
         *reinterpret_cast<uint32_t*>(sl + r * kVRow + c) = lo;
       }
     });
-    const int mt = warp & 3, nh = (warp >> 2) * 32;       // this warp's 16 x 32 part of the outputs
+    // this warp's 16 x 32 part of the outputs; the row tiles, whose causal work differs, rotate over the schedulers
+    const int mt = (warp + (warp >> 2)) & 3, nh = (warp >> 2) * 32;
     const int a_row = lane & 15, a_col = (lane >> 4) * 8;                          // fragments of A, row-major
     const int b_row = (lane & 7) + ((lane >> 4) & 1) * 8, b_col = ((lane >> 3) & 1) * 8;   // of B stored [n][k]
     const int bt_row = (lane & 7) + ((lane >> 3) & 1) * 8, bt_col = ((lane >> 4) & 1) * 8; // of B stored [k][n]
@@ -621,6 +623,7 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
         }
     }
     t0 += n;
+    base = t0 % kLinC ? make_float2(base.x + all.x, base.y + all.y) : make_float2(0.0f, 0.0f);
     if (STAGED) {
       buf ^= 1;
     } else if (t0 < t_end) {
@@ -634,7 +637,8 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
     if (r < dk && v0 + c < dv)
       *reinterpret_cast<float2*>(dst + (long long)r * dv + v0 + c) = make_float2(S[i][j][e], S[i][j][e + 1]);
   });
-  if (!OUT && v0 == 0 && part == 0 && ch < dk) *reinterpret_cast<float2*>(totals + seg * dk + ch) = total;
+  if (!OUT && v0 == 0 && part == 0 && ch < dk) *reinterpret_cast<float2*>(totals + seg * dk + ch) =
+        make_float2(expm1f(total.x * 0.6931471805599453f), expm1f(total.y * 0.6931471805599453f));
 }
 
 // ------------------------------------------------------------------------------------------- norm and gate
@@ -814,7 +818,7 @@ extern "C" int dptb_linear_attn(const DptbLinearArgs* a, void* stream_v) {
     if (a->dv % 4 == 0 && al16(a->state)) return a->f32 ? launch_step<float, 4>(p, st) : launch_step<__nv_bfloat16, 4>(p, st);
     return a->f32 ? launch_step<float, 1>(p, st) : launch_step<__nv_bfloat16, 1>(p, st);
   }
-  if (!dptb_linear_chunkable(a->dk, a->dv, a->f32)) return kErrUnsupported;
+  if (!dptb_linear_chunkable(a->dk, a->dv, a->f32) || a->q_scale <= 0.0f) return kErrUnsupported;
   if (a->ld % 8 || a->oq % 8 || a->ok % 8 || a->ov % 8 || !al16(a->log_a) || !al16(a->p) || !al16(a->state) || !al16(a->o)) return kErrBadShape;
   p.segments = a->segments < 1 ? 1 : a->segments;
   p.seg_tokens = linear_seg_tokens(a->S, p.segments);
@@ -826,11 +830,10 @@ extern "C" int dptb_linear_attn(const DptbLinearArgs* a, void* stream_v) {
   if (!a->decay) {
     if (!a->log_a) return kErrBadShape;
     p.log_a = a->log_a;
-    const size_t smem = (size_t)kDecayTokens * a->rank * sizeof(float);
-    const long long blocks = ((long long)a->B * a->S + kDecayTokens - 1) / kDecayTokens;
-    if (smem > 48 * 1024 || blocks > 0x7fffffff) return kErrTooLarge;
-    const int rc = counted(1, (int)launch_k(decay_kernel<__nv_bfloat16>, dim3((unsigned)blocks, (a->H * a->dk + 127) / 128),
-                                            dim3(128), smem, st, p));
+    const size_t smem = (size_t)kLinC * a->rank * sizeof(float);
+    if (smem > 48 * 1024) return kErrTooLarge;
+    const dim3 grid((a->S + kLinC - 1) / kLinC, (a->H * a->dk + 127) / 128, a->B);
+    const int rc = counted(1, (int)launch_k(decay_kernel<__nv_bfloat16>, grid, dim3(128), smem, st, p));
     if (rc) return rc;
   }
   const bool wide = linear_dv(a->dk, a->dv) == 128;
