@@ -244,7 +244,7 @@ __device__ __forceinline__ void lin_ldm_t(uint32_t (&r)[4], const __nv_bfloat16*
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
 }
 __device__ __forceinline__ void lin_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
       "{%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
@@ -274,8 +274,8 @@ struct LinSmem {
   static constexpr int kKBytes = kLinC * kKRow * 2;       // one part of the keys (or queries)
   static constexpr int kVBytes = kLinC * kVRow * 2;
   static constexpr int kSBytes = DK * kVRow * 2;
-  static constexpr int kK = 0;                            // [2][64][DK + 8] high, low; the scores [2][64][64 + 8] follow
-  static constexpr int kV = kK + 2 * (OUT && kPBytes > kKBytes ? kPBytes : kKBytes);
+  static constexpr int kK = 0;                            // [2][64][DK + 8] high, low; if not STAGED the scores take its place
+  static constexpr int kV = kK + 2 * kKBytes;
   static constexpr int kQ = kV + (kStaged ? 2 : 1) * kVBytes;   // pass 2 only from here
   static constexpr int kS = kQ + (OUT ? 2 * kKBytes : 0);
   static constexpr int kGate = kS + (OUT ? 2 * kSBytes : 0);
@@ -283,7 +283,9 @@ struct LinSmem {
   static constexpr int kRawK = kGate + 2 * DK * 4;
   static constexpr int kRawQ = kRawK + (kStaged ? kLinC * DK * 2 : 0);
   static constexpr int kRawA = kRawQ + (kStaged && OUT ? kLinC * DK * 2 : 0);
-  static constexpr int kTotal = kRawA + (kStaged ? kLinC * DK * 4 : 0);
+  static constexpr int kP = kStaged ? kRawA + kLinC * DK * 4 : kK;   // scores, [2][64][64 + 8]
+  static constexpr int kTotal = kStaged ? kP + (OUT ? 2 * kPBytes : 0) : kRawA;
+  static_assert(kStaged || kPBytes <= kKBytes, "the scores fit where the keys were");
   static_assert(kTotal <= 227 * 1024, "linear attention: shared memory budget");
 };
 
@@ -310,7 +312,7 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
   bf* ql = qh + kLinC * KR;
   bf* sh = reinterpret_cast<bf*>(lin_smem + L::kS);
   bf* sl = sh + DK * kVRow;
-  bf* ph = reinterpret_cast<bf*>(lin_smem + L::kK);
+  bf* ph = reinterpret_cast<bf*>(lin_smem + L::kP);
   bf* pl = ph + kLinC * kPRow;
   float* g_in = reinterpret_cast<float*>(lin_smem + L::kGate);  // factor on the state before the piece's products
   float* g_out = g_in + DK;                       // ... and after them
@@ -417,11 +419,10 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
   float2 total = make_float2(0.0f, 0.0f);         // of this thread's channels (threads with part == 0)
   float2 base = make_float2(0.0f, 0.0f);          // decay of the block before the piece
   int buf = 0;
-  if (t_begin < t_end) fetch(t_begin, 0);
-  for (int t0 = t_begin; t0 < t_end;) {
-    int n = min(kLinC - t0 % kLinC, t_end - t0);  // pieces do not cross blocks
+  // A fetch has arrived: this thread's copies of the values pass through their activation, in place.
+  auto arrived = [&](int buf) {
     lin_cp_wait();
-    if (p.silu) {               // this thread's own copies, in place
+    if (p.silu) {
       for (int i = tid; i < kLinC * DV / 8; i += NTHR) {
         uint4* at = reinterpret_cast<uint4*>(vs + buf * (kLinC * kVRow) + i / (DV / 8) * kVRow + i % (DV / 8) * 8);
         uint4 u = *at;
@@ -434,7 +435,14 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
         *at = u;
       }
     }
-    __syncthreads();            // the piece's rows are there, and everyone is done with the one before
+  };
+  if (t_begin < t_end) fetch(t_begin, 0);
+  arrived(0);
+  __syncthreads();
+  // Three barriers a piece in pass 2: everyone is done with the one before (and agrees on this one's length); operands are
+  // there; scores and the next piece's rows are there.  Two in pass 1: rows are there; operands are there.
+  for (int t0 = t_begin; t0 < t_end;) {
+    int n = min(kLinC - t0 % kLinC, t_end - t0);  // pieces do not cross blocks
     const bf* v_now = vs + buf * (kLinC * kVRow);
     // ---- a piece whose decays span too much becomes shorter
     auto decay_to = [&](int t) {
@@ -445,6 +453,7 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
       }
       return g;
     };
+    if (!OUT) __syncthreads();
     float2 all = decay_to(n - 1), first = make_float2(0.0f, 0.0f);
     if constexpr (OUT) {
       first = decay_to(0);
@@ -522,21 +531,35 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
           uint32_t ah[4], al[4];
           lin_ldm(ah, qh + (mt * 16 + a_row) * KR + kk * 16 + a_col);
           lin_ldm(al, ql + (mt * 16 + a_row) * KR + kk * 16 + a_col);
+          uint32_t bh4[NA / 2][4], bl4[NA / 2][4];
 #pragma unroll
           for (int j = 0; j < NA / 2; ++j) {
-            uint32_t bh4[4], bl4[4];
-            lin_ldm(bh4, kh + (na + j * 16 + b_row) * KR + kk * 16 + b_col);
-            lin_ldm(bl4, kl + (na + j * 16 + b_row) * KR + kk * 16 + b_col);
-#pragma unroll
-            for (int x = 0; x < 2; ++x) {
-              lin_mma(a[j * 2 + x], ah, bh4[2 * x], bh4[2 * x + 1]);
-              lin_mma(a[j * 2 + x], ah, bl4[2 * x], bl4[2 * x + 1]);
-              lin_mma(a[j * 2 + x], al, bh4[2 * x], bh4[2 * x + 1]);
-            }
+            lin_ldm(bh4[j], kh + (na + j * 16 + b_row) * KR + kk * 16 + b_col);
+            lin_ldm(bl4[j], kl + (na + j * 16 + b_row) * KR + kk * 16 + b_col);
           }
+          // neighbouring products go to different accumulators
+#pragma unroll
+          for (int j = 0; j < NA; ++j) lin_mma(a[j], ah, bh4[j / 2][j % 2 * 2], bh4[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+          for (int j = 0; j < NA; ++j) lin_mma(a[j], ah, bl4[j / 2][j % 2 * 2], bl4[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+          for (int j = 0; j < NA; ++j) lin_mma(a[j], al, bh4[j / 2][j % 2 * 2], bh4[j / 2][j % 2 * 2 + 1]);
         }
       }
     }
+    auto put_scores = [&]() {
+#pragma unroll
+      for (int j = 0; j < NA; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = na + j * 8 + (lane & 3) * 2;
+          uint32_t hi, lo;
+          split_pair(c <= r ? a[j][e] : 0.0f, c + 1 <= r ? a[j][e + 1] : 0.0f, hi, lo);
+          *reinterpret_cast<uint32_t*>(ph + r * kPRow + c) = hi;
+          *reinterpret_cast<uint32_t*>(pl + r * kPRow + c) = lo;
+        }
+    };
+    if (OUT && STAGED) put_scores();
     // ---- the state after the piece
 #pragma unroll
     for (int kk = 0; kk < kLinC / 16; ++kk) {
@@ -549,10 +572,9 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
         lin_ldm_t(ah, kh + (kk * 16 + b_row) * KR + m0 + i * 16 * WARPS + b_col);
         lin_ldm_t(al, kl + (kk * 16 + b_row) * KR + m0 + i * 16 * WARPS + b_col);
 #pragma unroll
-        for (int j = 0; j < NT; ++j) {
-          lin_mma(S[i][j], ah, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
-          lin_mma(S[i][j], al, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
-        }
+        for (int j = 0; j < NT; ++j) lin_mma(S[i][j], ah, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) lin_mma(S[i][j], al, vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
       }
     }
     if constexpr (OUT) {
@@ -561,17 +583,11 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
         S[i][j][e] *= g;
         S[i][j][e + 1] *= g;
       });
-      __syncthreads();          // the keys are done with: the scores take their place
-#pragma unroll
-      for (int j = 0; j < NA; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = na + j * 8 + (lane & 3) * 2;
-          uint32_t hi, lo;
-          split_pair(c <= r ? a[j][e] : 0.0f, c + 1 <= r ? a[j][e + 1] : 0.0f, hi, lo);
-          *reinterpret_cast<uint32_t*>(ph + r * kPRow + c) = hi;
-          *reinterpret_cast<uint32_t*>(pl + r * kPRow + c) = lo;
-        }
+      if (!STAGED) {
+        __syncthreads();        // the keys are done with: the scores take their place
+        put_scores();
+      }
+      if (STAGED && t0 + n < t_end) arrived(buf ^ 1);
       __syncthreads();
       // ---- outputs: own tokens, then everything before the piece
       float o[4][4];
@@ -583,34 +599,31 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
         uint32_t ah[4], al[4];
         lin_ldm(ah, ph + (mt * 16 + a_row) * kPRow + kk * 16 + a_col);
         lin_ldm(al, pl + (mt * 16 + a_row) * kPRow + kk * 16 + a_col);
+        uint32_t vb[2][4];
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          uint32_t vb[4];
-          lin_ldm_t(vb, v_now + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
+        for (int j = 0; j < 2; ++j) lin_ldm_t(vb[j], v_now + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
 #pragma unroll
-          for (int x = 0; x < 2; ++x) {
-            lin_mma(o[j * 2 + x], ah, vb[2 * x], vb[2 * x + 1]);
-            lin_mma(o[j * 2 + x], al, vb[2 * x], vb[2 * x + 1]);
-          }
-        }
+        for (int j = 0; j < 4; ++j) lin_mma(o[j], ah, vb[j / 2][j % 2 * 2], vb[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) lin_mma(o[j], al, vb[j / 2][j % 2 * 2], vb[j / 2][j % 2 * 2 + 1]);
       }
 #pragma unroll
       for (int kk = 0; kk < DK / 16; ++kk) {
         uint32_t ah[4], al[4];
         lin_ldm(ah, qh + (mt * 16 + a_row) * KR + kk * 16 + a_col);
         lin_ldm(al, ql + (mt * 16 + a_row) * KR + kk * 16 + a_col);
+        uint32_t bh4[2][4], bl4[2][4];
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          uint32_t bh4[4], bl4[4];
-          lin_ldm_t(bh4, sh + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
-          lin_ldm_t(bl4, sl + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
-#pragma unroll
-          for (int x = 0; x < 2; ++x) {
-            lin_mma(o[j * 2 + x], ah, bh4[2 * x], bh4[2 * x + 1]);
-            lin_mma(o[j * 2 + x], ah, bl4[2 * x], bl4[2 * x + 1]);
-            lin_mma(o[j * 2 + x], al, bh4[2 * x], bh4[2 * x + 1]);
-          }
+          lin_ldm_t(bh4[j], sh + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
+          lin_ldm_t(bl4[j], sl + (kk * 16 + bt_row) * kVRow + nh + j * 16 + bt_col);
         }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) lin_mma(o[j], ah, bh4[j / 2][j % 2 * 2], bh4[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) lin_mma(o[j], ah, bl4[j / 2][j % 2 * 2], bl4[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) lin_mma(o[j], al, bh4[j / 2][j % 2 * 2], bh4[j / 2][j % 2 * 2 + 1]);
       }
       bf* out = static_cast<bf*>(p.o) + (row_b + t0) * p.H * dv + (long long)h * dv + v0;
 #pragma unroll
@@ -625,10 +638,13 @@ __global__ void __launch_bounds__(kLinThreads * DV, DK <= 64 && DV <= 64 ? 2 : 1
     t0 += n;
     base = t0 % kLinC ? make_float2(base.x + all.x, base.y + all.y) : make_float2(0.0f, 0.0f);
     if (STAGED) {
+      if (!OUT && t0 < t_end) arrived(buf ^ 1);
       buf ^= 1;
     } else if (t0 < t_end) {
       __syncthreads();
       fetch(t0, 0);
+      arrived(0);
+      __syncthreads();
     }
   }
   if (OUT && seg != p.segments - 1) return;
