@@ -95,6 +95,7 @@ def _rows(p: torch.Tensor, rows: int, cols: int, what: str) -> int:
 
 # --------------------------------------------------------------------------- linear attention
 CHUNK_ROWS = 16       # tokens per sequence from which the tensor-core form runs
+MAX_CHUNK_RANK = 192  # of the low-rank decay in that form (shared memory of the kernel that sums the decays)
 
 
 def linear_chunkable(dk: int, dv: int, f32: bool) -> bool:
@@ -125,7 +126,8 @@ def linear_attn(p: torch.Tensor, cols: dict, state: torch.Tensor, B: int, S: int
     a.o = o.data_ptr()
     a.B, a.S, a.H, a.dk, a.dv, a.silu, a.f32, a.q_scale = B, S, H, dk, dv, int(silu), f32, q_scale
     if chunked is None:
-        chunked = S >= CHUNK_ROWS and linear_chunkable(dk, dv, bool(f32)) and a.ld % 8 == 0 and p.data_ptr() % 16 == 0
+        chunked = S >= CHUNK_ROWS and linear_chunkable(dk, dv, bool(f32)) and a.ld % 8 == 0 and p.data_ptr() % 16 == 0 and \
+            a.rank <= MAX_CHUNK_RANK and q_scale > 0.0
     a.chunked = int(chunked)
     if chunked:
         a.segments = _lib().dptb_linear_segments(B, S, H, dk, dv) if segments is None else segments

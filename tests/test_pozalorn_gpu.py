@@ -84,7 +84,7 @@ def run_linear(cols, p, state, B, T, cut, H, dk, dv, **kw):
 
 @pytest.mark.parametrize("dtype", [F32, BF])
 @pytest.mark.parametrize("H,dk,dv,rank", [(1, 8, 8, 1), (3, 16, 24, 5), (2, 32, 64, 16), (2, 48, 136, 3), (1, 64, 40, 7),
-                                          (2, 128, 72, 4), (1, 200, 64, 16), (3, 12, 6, 9), (1, 256, 128, 2), (2, 33, 16, 4)])
+                                          (2, 128, 72, 4), (1, 200, 64, 16), (2, 64, 128, 200), (3, 12, 6, 9), (1, 256, 128, 2), (2, 33, 16, 4)])
 def test_gated_linear_attention(dtype, H, dk, dv, rank):
     B, T, tau, qs = 2, 150, 4.0, 0.3
     cols, p, w2, b2 = linear_case(dtype, B, T, H, dk, dv, rank, 2.0)
