@@ -40,16 +40,27 @@ struct PrepParams {
 
 constexpr int kPrepThreads = 256;
 
-// The mean of the block of `pool` rows that starts at position p0, feature c.
-template <typename T>
-__device__ __forceinline__ float block_mean(const T* rows, long long ld, int c, int p0, int pool, int ring, int lin0) {
-  float s = 0.0f;
-  int at = ring ? p0 % ring : p0 - lin0;
+// The mean of the block of `pool` rows that starts at position p0, features c ... c + V - 1.
+template <typename T, int V>
+__device__ __forceinline__ void block_mean(const T* rows, long long ld, int c, int p0, int pool, int ring, int lin0, T* out) {
+  float s[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) s[e] = 0.0f;
+  const int start = ring ? p0 % ring : p0 - lin0;
+#pragma unroll 8
   for (int j = 0; j < pool; ++j) {
-    s += to_f32(rows[(long long)at * ld + c]);
-    if (++at == ring) at = 0;
+    const int at = ring && start + j >= ring ? start + j - ring : start + j;
+    const T* r = rows + at * ld + c;
+    float v[V];
+    if constexpr (V == 8) Vec8<T>::load(r, v);
+    else v[0] = to_f32(r[0]);
+#pragma unroll
+    for (int e = 0; e < V; ++e) s[e] += v[e];
   }
-  return s / (float)pool;
+#pragma unroll
+  for (int e = 0; e < V; ++e) s[e] /= (float)pool;
+  if constexpr (V == 8) Vec8<T>::store(out, s);
+  else out[0] = from_f32<T>(s[0]);
 }
 
 // One CTA per token.  Rows are staged in shared memory as fp32; V consecutive features per thread and access.
@@ -179,12 +190,10 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prep_kernel(const PrepParams
     const int blk = pos / p.pool - 1;
     const T* kr = static_cast<const T*>(p.k_ring) + (long long)b * p.ring * nk;
     const T* vr = static_cast<const T*>(p.v_ring) + (long long)b * p.ring * nv;
-    for (int c = tid; c < nk; c += kPrepThreads)
-      static_cast<T*>(p.k_pool)[((long long)b * p.pool_rows + blk) * nk + c] =
-          from_f32<T>(block_mean(kr, nk, c, blk * p.pool, p.pool, p.ring, 0));
-    for (int c = tid; c < nv; c += kPrepThreads)
-      static_cast<T*>(p.v_pool)[((long long)b * p.pool_rows + blk) * nv + c] =
-          from_f32<T>(block_mean(vr, nv, c, blk * p.pool, p.pool, p.ring, 0));
+    T* kp = static_cast<T*>(p.k_pool) + ((long long)b * p.pool_rows + blk) * nk;
+    T* vp = static_cast<T*>(p.v_pool) + ((long long)b * p.pool_rows + blk) * nv;
+    for (int c = tid * V; c < nk; c += kPrepThreads * V) block_mean<T, V>(kr, nk, c, blk * p.pool, p.pool, p.ring, 0, kp + c);
+    for (int c = tid * V; c < nv; c += kPrepThreads * V) block_mean<T, V>(vr, nv, c, blk * p.pool, p.pool, p.ring, 0, vp + c);
   }
 }
 
@@ -197,18 +206,21 @@ struct PoolParams {
   int nk, nv, ring, lin0, pool, pool_rows, first;   // blocks first + blockIdx.x
 };
 
-template <typename T>
-__global__ void __launch_bounds__(256) pool_blocks_kernel(const PoolParams p) {
+constexpr int kPoolThreads = 128;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kPoolThreads) pool_blocks_kernel(const PoolParams p) {
   const int blk = p.first + blockIdx.x, b = blockIdx.y;
   pdl_wait();
   pdl_launch_dependents();
   const T* k = static_cast<const T*>(p.k) + b * p.k_batch;
   const T* v = static_cast<const T*>(p.v) + b * p.v_batch;
-  const long long out = (long long)b * p.pool_rows + blk;
-  for (int c = threadIdx.x; c < p.nk; c += 256)
-    static_cast<T*>(p.k_pool)[out * p.nk + c] = from_f32<T>(block_mean(k, p.nk, c, blk * p.pool, p.pool, p.ring, p.lin0));
-  for (int c = threadIdx.x; c < p.nv; c += 256)
-    static_cast<T*>(p.v_pool)[out * p.nv + c] = from_f32<T>(block_mean(v, p.nv, c, blk * p.pool, p.pool, p.ring, p.lin0));
+  T* kp = static_cast<T*>(p.k_pool) + ((long long)b * p.pool_rows + blk) * p.nk;
+  T* vp = static_cast<T*>(p.v_pool) + ((long long)b * p.pool_rows + blk) * p.nv;
+  for (int c = threadIdx.x * V; c < p.nk + p.nv; c += kPoolThreads * V) {
+    if (c < p.nk) block_mean<T, V>(k, p.nk, c, blk * p.pool, p.pool, p.ring, p.lin0, kp + c);
+    else block_mean<T, V>(v, p.nv, c - p.nk, blk * p.pool, p.pool, p.ring, p.lin0, vp + c - p.nk);
+  }
 }
 
 struct WindowParams {
@@ -361,7 +373,7 @@ extern "C" int dptb_qkv_prep(const DptbPrepArgs* a, void* stream_v) {
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   bool vec = a->dk % 8 == 0 && a->dv % 8 == 0 && a->ld % 8 == 0 && a->oq % 8 == 0 && a->ok % 8 == 0 && a->ov % 8 == 0;
   for (const void* q : {a->p, (const void*)a->q, (const void*)a->k_ring, (const void*)a->v_ring, (const void*)a->k_lin,
-                        (const void*)a->v_lin, a->gq, a->gk})
+                        (const void*)a->v_lin, a->gq, a->gk, (const void*)a->k_pool, (const void*)a->v_pool})
     vec = vec && al16(q);
   const size_t smem = ((size_t)(a->H + a->G) * (a->dk + 1)) * sizeof(float);
   if (smem > 200 * 1024) return kErrTooLarge;
@@ -387,8 +399,12 @@ extern "C" int dptb_pool_blocks(const DptbPoolArgs* a, void* stream_v) {
   p.nk = a->nk; p.nv = a->nv; p.ring = a->ring; p.lin0 = a->lin0; p.pool = a->pool; p.pool_rows = a->pool_rows;
   p.first = a->first;
   const dim3 grid(a->count, a->B);
-  return counted(1, (int)(a->f32 ? launch_k(pool_blocks_kernel<float>, grid, dim3(256), (size_t)0, st, p)
-                                 : launch_k(pool_blocks_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)0, st, p)));
+  bool vec = a->nk % 8 == 0 && a->nv % 8 == 0 && a->k_batch % 8 == 0 && a->v_batch % 8 == 0;
+  for (const void* q : {a->k, a->v, (const void*)a->k_pool, (const void*)a->v_pool})
+    vec = vec && (reinterpret_cast<uintptr_t>(q) & 15) == 0;
+  auto kern = a->f32 ? (vec ? pool_blocks_kernel<float, 8> : pool_blocks_kernel<float, 1>)
+                     : (vec ? pool_blocks_kernel<__nv_bfloat16, 8> : pool_blocks_kernel<__nv_bfloat16, 1>);
+  return counted(1, (int)launch_k(kern, grid, dim3(kPoolThreads), (size_t)0, st, p));
 }
 
 struct DptbWindowArgs {
