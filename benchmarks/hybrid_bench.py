@@ -53,7 +53,7 @@ def famudra_config(s) -> dict:
 
 
 def pozalorn_config(s) -> dict:
-    rot = {"base": 500000.0, "dims": s["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    rot = {"base": 1e6, "dims": s["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
     att = dict(heads=s["heads"], kv_heads=max(1, s["heads"] // 4), dim=s["dim"], vdim=s["dim"], rot=rot, scale=s["dim"] ** -0.5)
     lin = dict(heads=s["lin_heads"], dim=s["lin_dim"], vdim=s["lin_vdim"])
     mixers = [("gla", dict(lin, tau=16.0)),

@@ -114,7 +114,7 @@ def test_row_layout_is_aligned():
 
 
 @pytest.mark.parametrize("scaling", [None, SCALING, {"factor": 2.0, "low": 0.5, "high": 20.0, "original": 100}])
-@pytest.mark.parametrize("base,dims", [(10000.0, 16), (500.0, 6), (20000.0, 64)])
+@pytest.mark.parametrize("base,dims", [(10000.0, 16), (500.0, 6), (30000.0, 48)])
 def test_rotary_table(scaling, base, dims):
     t = RotaryTable(base, dims, scaling)
     f = oracle.frequencies({"base": base, "dims": dims, "scaling": scaling})
